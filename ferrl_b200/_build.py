@@ -21,6 +21,7 @@ ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 CSRC = os.path.join(ROOT, "csrc")
 BUILD = os.path.join(ROOT, "build")
 SO_PATH = os.path.join(ROOT, "ferrl_b200", "_C.so")
+SO_STAMP = os.path.join(ROOT, "ferrl_b200", "bin", "_C.sources")     # what the library in the tree was built from
 LAUNCHER_SRC = os.path.join(CSRC, "native", "sandbox_launcher.cpp")
 LAUNCHER_BIN = os.path.join(ROOT, "ferrl_b200", "bin", "ferrl-sandbox-launch")
 
@@ -72,7 +73,28 @@ def build_io(force: bool = False) -> str:
     return IO_LIB
 
 
-def build(force: bool = False, verbose: bool = False) -> str:
+def _source_key() -> str:
+    """Hash of everything the library is compiled from (contents and relative names), flags and torch version."""
+    import torch
+    h = hashlib.sha256((" ".join(NVCC_FLAGS) + torch.__version__).encode())
+    for p in sorted(glob.glob(os.path.join(CSRC, "**", "*"), recursive=True)):
+        if p.endswith((".cu", ".cuh", ".cpp", ".h")) and os.sep + "native" + os.sep not in p:
+            with open(p, "rb") as f:
+                h.update(os.path.relpath(p, ROOT).encode() + b"\0" + f.read())
+    return h.hexdigest()
+
+
+def ensure() -> str:
+    """Build the library unless the one in the tree was made from these very sources (a checkout that came with its
+    library compiles nothing, a fresh one everything but the sandbox launcher)."""
+    have = ""
+    if os.path.exists(SO_PATH) and os.path.exists(SO_STAMP):
+        with open(SO_STAMP) as f:
+            have = f.read()
+    return SO_PATH if have == _source_key() else build(launcher=False)
+
+
+def build(force: bool = False, verbose: bool = False, launcher: bool = True) -> str:
     import torch
     from torch.utils import cpp_extension as ce
     os.makedirs(BUILD, exist_ok=True)
@@ -81,7 +103,8 @@ def build(force: bool = False, verbose: bool = False) -> str:
     cu = sorted(glob.glob(os.path.join(CSRC, "**", "*.cu"), recursive=True))
     cpp = sorted(p for p in glob.glob(os.path.join(CSRC, "**", "*.cpp"), recursive=True)
                  if os.sep + "native" + os.sep not in p)   # csrc/native holds standalone host programs
-    build_launcher(force)
+    if launcher:
+        build_launcher(force)
     build_io(force)
     nvcc = _nvcc()
     cuda_home = os.path.dirname(os.path.dirname(nvcc))
@@ -119,6 +142,8 @@ def build(force: bool = False, verbose: bool = False) -> str:
         _run(link)
         with open(stamp, "w") as f:
             f.write(want)
+    with open(SO_STAMP, "w") as f:
+        f.write(_source_key())
     keep = {os.path.basename(o) for o in objs}
     for name in os.listdir(BUILD):   # objects of earlier source versions
         base = name[:-4] if name.endswith(".log") else name

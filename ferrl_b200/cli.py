@@ -9,6 +9,8 @@ Verbs (reference ``crates/ferrl/src/bin/ferrl.rs:116-131``):
     perf-gate         compare a candidate run's metrics stream against a baseline's
     trimul-baseline   time the reference kernel to pin ``trimul.baseline.ns``
     verifier-executor serve the dedicated-UID verifier socket
+    generate          token ids in, sampled or greedy continuations out (any model family)
+    trace             feed a token trace through a model and write chosen logits (also ``bin/trace_run``)
 
 The reference verb names are accepted as aliases.  Multi-GPU launches use one
 process per GPU (``torchrun`` or Slurm ``srun`` with ``FERRL_NCCL_RENDEZVOUS``);
@@ -350,6 +352,33 @@ def cmd_verifier_executor(args) -> int:
     return 0
 
 
+def cmd_generate(args) -> int:
+    """Continuations of the prompts on standard input, one JSON list of token ids a line; one JSON list of new tokens
+    a line comes out, in the same order."""
+    import torch
+    from .lm_policy import LmPolicy
+    from .models.loader import LoaderOpts, load_auto_policy
+    from .policy import EvalSampling, GenConfig
+    from .sampler import GrpoSampler
+    from .trace import DTYPES
+    prompts = [json.loads(line) for line in sys.stdin if line.strip()]
+    model, _ = load_auto_policy(args.model, LoaderOpts(dtype=DTYPES[args.dtype], device=args.device, lora=None))
+    # greedy decoding is the nucleus that holds nothing but the most probable token
+    sampling = EvalSampling(args.temperature, 1e-9 if args.greedy else args.top_p)
+    cfg = GenConfig(group_size=1, max_new_tokens=args.max_new_tokens, eos_token_id=args.eos, eval_sampling=sampling)
+    policy = LmPolicy(model, GrpoSampler(args.seed))
+    with torch.no_grad():
+        outs = policy.generate_batch(prompts, cfg, list(range(len(prompts))))
+    for r in outs:
+        print(json.dumps(r.completion(0)))
+    return 0
+
+
+def cmd_trace(args) -> int:
+    from . import trace
+    return trace.run(args)
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="ferrl-b200")
     sub = ap.add_subparsers(dest="verb", required=True)
@@ -420,6 +449,21 @@ def main(argv=None) -> int:
     p.add_argument("--client-uid", type=int, required=True, help="the only UID whose requests are served")
     p.add_argument("--socket-mode", type=lambda v: int(v, 8), default=0o660)
     p.set_defaults(fn=cmd_verifier_executor)
+    p = sub.add_parser("generate")
+    p.add_argument("--model", required=True, help="folder with config.json and safetensors weights")
+    p.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
+    p.add_argument("--device", default="cuda")
+    p.add_argument("--max-new-tokens", type=int, default=64)
+    p.add_argument("--greedy", action="store_true")
+    p.add_argument("--temperature", type=float, default=1.0)
+    p.add_argument("--top-p", type=float, default=None)
+    p.add_argument("--seed", type=int, default=0)
+    p.add_argument("--eos", type=int, default=None)
+    p.set_defaults(fn=cmd_generate)
+    p = sub.add_parser("trace")
+    from .trace import add_arguments
+    add_arguments(p)
+    p.set_defaults(fn=cmd_trace)
     args = ap.parse_args(argv)
     return args.fn(args)
 

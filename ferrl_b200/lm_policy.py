@@ -86,6 +86,40 @@ class LmPolicy(Policy):
         return self.sampler.temperature, validate_top_p(cfg.top_p)
 
     # ------------------------------------------------------------- rollout
+    def pack_prompts(self, prompts: Sequence[Sequence[int]]):
+        """``(ids [P, Lmax] right-padded, lens [P])`` on the model's device."""
+        dev = self.device()
+        lens_host = torch.tensor([len(p) for p in prompts], dtype=torch.int64)
+        ids_host = torch.full((len(prompts), int(lens_host.max())), self.pad_token_id, dtype=torch.int64)
+        for i, p in enumerate(prompts):
+            ids_host[i, :len(p)] = torch.as_tensor(list(p), dtype=torch.int64)
+        if dev.type == "cuda":
+            ids_host, lens_host = ids_host.pin_memory(), lens_host.pin_memory()
+        self.h2d_bytes += ids_host.numel() * 8 + lens_host.numel() * 8
+        return ids_host.to(dev, non_blocking=True), lens_host.to(dev, non_blocking=True)
+
+    def refresh_merged(self) -> None:
+        if not self._merged_fresh:
+            self.model.merge_adapters()
+            self._merged_fresh = True
+
+    def decoder_for(self, batch: int, max_len: int, group: int = 1):
+        """``(decoder, its key)`` for ``batch`` rows of up to ``max_len`` tokens; the last one is kept and reused."""
+        if self.device().type == "cuda":
+            max_len = (max_len + 127) // 128 * 128  # bucket the cache length so decoders and graphs are reused
+        key = (batch, max_len, group)
+        dec = self._decoders.get(key)
+        if dec is None:
+            self._decoders.clear()
+            self._graphs.clear()
+            try:
+                dec = self.model.new_decoder(batch, max_len, self.comm, group=group)
+            except TypeError:       # model families whose decoder takes no group argument
+                dec = self.model.new_decoder(batch, max_len, self.comm)
+            self._decoders[key] = dec
+        self.last_cache_bytes = dec.cache_bytes()
+        return dec, key
+
     @torch.no_grad()
     def generate_batch(self, prompts: Sequence[Sequence[int]], cfg: GenConfig,
                        global_row_bases: Sequence[int]) -> list[Rollout]:
@@ -99,35 +133,12 @@ class LmPolicy(Policy):
         dev = self.device()
         P, G, N = len(prompts), cfg.group_size, cfg.max_new_tokens
         B = P * G
-        lens_host = torch.tensor([len(p) for p in prompts], dtype=torch.int64)
-        Lmax = int(lens_host.max())
-        ids_host = torch.full((P, Lmax), self.pad_token_id, dtype=torch.int64)
-        for i, p in enumerate(prompts):
-            ids_host[i, :len(p)] = torch.as_tensor(list(p), dtype=torch.int64)
-        if dev.type == "cuda":
-            ids_host, lens_host = ids_host.pin_memory(), lens_host.pin_memory()
-        ids = ids_host.to(dev, non_blocking=True)
-        lens = lens_host.to(dev, non_blocking=True)
-        self.h2d_bytes += ids_host.numel() * 8 + lens_host.numel() * 8 + B * 8
+        ids, lens = self.pack_prompts(prompts)
+        self.h2d_bytes += B * 8
         rows = (torch.as_tensor(list(global_row_bases), dtype=torch.int64).repeat_interleave(G)
                 + torch.arange(G, dtype=torch.int64).repeat(P)).to(dev)
-        if not self._merged_fresh:
-            self.model.merge_adapters()
-            self._merged_fresh = True
-        max_len = Lmax + N
-        if dev.type == "cuda":
-            max_len = (max_len + 127) // 128 * 128  # bucket the cache length so decoders and graphs are reused
-        dkey = (B, max_len, G)
-        dec = self._decoders.get(dkey)
-        if dec is None:
-            self._decoders.clear()
-            self._graphs.clear()
-            try:
-                dec = self.model.new_decoder(B, max_len, self.comm, group=G)
-            except TypeError:       # model families whose decoder takes no group argument
-                dec = self.model.new_decoder(B, max_len, self.comm)
-            self._decoders[dkey] = dec
-        self.last_cache_bytes = dec.cache_bytes()
+        self.refresh_merged()
+        dec, (_, max_len, _) = self.decoder_for(B, ids.shape[1] + N, G)
         logits = dec.prefill(ids, lens)
         dec.broadcast_groups(G)
         logits = logits.repeat_interleave(G, dim=0)

@@ -473,9 +473,11 @@ class DenseCachedDecoder:
         return sum(t.numel() * t.element_size() for t in self.k + self.v)
 
     @torch.no_grad()
-    def prefill(self, ids: torch.Tensor, lens: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    def prefill(self, ids: torch.Tensor, lens: torch.Tensor, rows: Optional[torch.Tensor] = None,
+                at: Optional[tuple] = None) -> torch.Tensor:
         """Prefill ``ids`` ``[P, L]`` (right-padded, true lengths ``lens``) into
-        cache rows ``rows`` (default ``0..P``); returns last-token logits ``[P, V]``."""
+        cache rows ``rows`` (default ``0..P``); returns last-token logits ``[P, V]``, or those of the
+        places ``at = (prompt indices, positions)``."""
         m = self.m
         P, L = ids.shape
         rows = torch.arange(P, device=ids.device) if rows is None else rows
@@ -487,7 +489,7 @@ class DenseCachedDecoder:
             self.k[i][rows, :L] = tmp[i][0]
             self.v[i][rows, :L] = tmp[i][1]
         self.kv_len[rows] = lens.to(torch.int32)
-        last = h[torch.arange(P, device=ids.device), (lens - 1).long()]
+        last = h[(torch.arange(P, device=ids.device), (lens - 1).long()) if at is None else at]
         last = ops.rmsnorm(last, m.final_norm, m.spec.rms_norm_eps)
         return ops.lora_linear(last, m.head_weight(), None, None).float()
 
@@ -587,7 +589,8 @@ class DensePagedDecoder(DenseCachedDecoder):
         return (self.prefix_len, self.group) if self.share_prefix else None
 
     @torch.no_grad()
-    def prefill(self, ids: torch.Tensor, lens: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
+    def prefill(self, ids: torch.Tensor, lens: torch.Tensor, rows: Optional[torch.Tensor] = None,
+                at: Optional[tuple] = None) -> torch.Tensor:
         """Prefill the ``P = batch // group`` prompts; afterwards every row ``p*group + g`` sees its
         prompt (``broadcast_groups`` has nothing left to copy)."""
         if rows is not None:
@@ -621,7 +624,7 @@ class DensePagedDecoder(DenseCachedDecoder):
                 tail = torch.gather(src, 1, tail_idx[:, :, None, None].expand(P, page, hkv, D))
                 pool[first_private] = tail.repeat_interleave(G, dim=0)
         self.kv_len.copy_(lens.to(torch.int32).repeat_interleave(G))
-        last = h[torch.arange(P, device=dev), (lens - 1).long()]
+        last = h[(torch.arange(P, device=dev), (lens - 1).long()) if at is None else at]
         last = ops.rmsnorm(last, m.final_norm, m.spec.rms_norm_eps)
         return ops.lora_linear(last, m.head_weight(), None, None).float()
 

@@ -407,7 +407,7 @@ class Gemma4CachedDecoder:
         return sum(2 * k.shape[0] * self.max_len * k.shape[2] * k.shape[3] * k.element_size() for k in self.k)
 
     @torch.no_grad()
-    def prefill(self, ids, lens, rows=None):
+    def prefill(self, ids, lens, rows=None, at=None):
         m = self.m
         P, L = ids.shape
         rows = torch.arange(P, device=ids.device) if rows is None else rows
@@ -427,7 +427,7 @@ class Gemma4CachedDecoder:
             self.k[i][rows] = torch.gather(tmp[i][0], 1, gi)
             self.v[i][rows] = torch.gather(tmp[i][1], 1, gi)
         self.kv_len[rows] = lens.to(torch.int32)
-        last = h[torch.arange(P, device=ids.device), (lens - 1).long()]
+        last = h[(torch.arange(P, device=ids.device), (lens - 1).long()) if at is None else at]
         last = ops.rmsnorm(last, m.final_norm, m.spec.rms_norm_eps)
         return m._softcap(ops.lora_linear(last, m.embed, None, None).float())
 

@@ -208,7 +208,7 @@ def read_config(model_dir: str) -> dict:
 def _identity(model_dir: str, cfg: dict, src: TensorSource, opts: Optional["LoaderOpts"] = None) -> PolicyLoadIdentity:
     with open(os.path.join(model_dir, "config.json"), "rb") as f:
         csha = hashlib.sha256(f.read()).hexdigest()
-    return PolicyLoadIdentity(str(cfg.get("model_type")), csha, src.files_sha256(),
+    return PolicyLoadIdentity(str(model_kind(cfg)), csha, src.files_sha256(),
                               execution_recipe(opts) if opts is not None else "")
 
 
@@ -232,15 +232,22 @@ def load_dense(model_dir: str, spec_fn: Callable[[dict], DenseSpec], opts: Loade
     return model, _identity(model_dir, cfg, src, opts)
 
 
+def model_kind(cfg: dict) -> Optional[str]:
+    """The key a configuration is dispatched on: ``model_type``, or ``architecture`` where there is none."""
+    kind = cfg.get("model_type")
+    return cfg.get("architecture") if kind is None else kind
+
+
 def load_auto_policy(model_dir: str, opts: Optional[LoaderOpts] = None):
     """Build the right model family from ``config.json`` and return
     ``(model, PolicyLoadIdentity)``.  ``model_type`` dispatch: ``qwen3`` ->
     dense Qwen3, ``qwen3_5``/``qwen3_5_text``/``qwen3_5_moe`` -> hybrid,
-    ``gemma4``/``gemma4_text`` -> Gemma.  Llama must be loaded explicitly with
+    ``gemma4``/``gemma4_text`` -> Gemma; ``architecture`` ``Galodra`` ->
+    latent attention with gated residuals.  Llama must be loaded explicitly with
     ``load_llama`` (library API only)."""
     opts = opts or LoaderOpts()
     cfg = read_config(model_dir)
-    mt = cfg.get("model_type")
+    mt = model_kind(cfg)
     if mt == "qwen3":
         from .qwen3 import qwen3_spec
         return load_dense(model_dir, qwen3_spec, opts)
@@ -250,7 +257,10 @@ def load_auto_policy(model_dir: str, opts: Optional[LoaderOpts] = None):
     if mt in ("gemma4", "gemma4_text", "gemma4_uni"):
         from .gemma4 import load_gemma4
         return load_gemma4(model_dir, opts)
-    raise ValueError(f"unsupported model_type {mt!r} (supported: qwen3, qwen3_5[_moe], gemma4)")
+    if mt == "Galodra":
+        from .galodra import load_galodra
+        return load_galodra(model_dir, opts)
+    raise ValueError(f"unsupported model_type {mt!r} (supported: qwen3, qwen3_5[_moe], gemma4, Galodra)")
 
 
 def load_llama(model_dir: str, opts: Optional[LoaderOpts] = None):

@@ -28,14 +28,20 @@ def ops_native(t):
     return ops.native(t)
 
 
-def topk_router(x: torch.Tensor, weight: torch.Tensor, top_k: int, renorm: bool = True):
-    """``x`` ``[T, H]``, router ``weight`` ``[E, H]`` -> ``(probs [T,E] f32, scores [T,k] f32, indices [T,k])``."""
-    logits = F.linear(x, weight)
-    probs = torch.softmax(logits.float(), dim=-1)
+def topk_scores(logits: torch.Tensor, top_k: int, renorm: bool = True, score: str = "softmax"):
+    """Router ``logits`` ``[T, E]`` -> ``(probs [T,E] f32, scores [T,k] f32, indices [T,k])``.  ``score`` turns logits
+    into scores: ``softmax`` over the experts, or ``sigmoid`` of each expert by itself."""
+    z = logits.float()
+    probs = torch.softmax(z, dim=-1) if score == "softmax" else torch.sigmoid(z)
     scores, idx = torch.topk(probs, top_k, dim=-1)
     if renorm:
         scores = scores / scores.sum(-1, keepdim=True)
     return probs, scores, idx
+
+
+def topk_router(x: torch.Tensor, weight: torch.Tensor, top_k: int, renorm: bool = True):
+    """``x`` ``[T, H]``, router ``weight`` ``[E, H]`` -> ``(probs [T,E] f32, scores [T,k] f32, indices [T,k])``."""
+    return topk_scores(F.linear(x, weight), top_k, renorm)
 
 
 @dataclass
@@ -75,16 +81,33 @@ def grouped_swiglu(xs: torch.Tensor, offsets: torch.Tensor, gate_up: torch.Tenso
 
 
 def moe_experts(x: torch.Tensor, indices: torch.Tensor, scores: torch.Tensor, gate_up: torch.Tensor,
-                down: torch.Tensor, act: str = "silu") -> torch.Tensor:
-    """Routed experts: permute -> grouped SwiGLU -> weight -> scatter-add. ``x`` ``[T,H]``."""
+                down: torch.Tensor, act: str = "silu", weight_input: bool = False) -> torch.Tensor:
+    """Routed experts: permute -> grouped SwiGLU -> weight -> scatter-add. ``x`` ``[T,H]``.  With ``weight_input`` the
+    routing weight multiplies an expert's input instead of its output."""
     E = gate_up.shape[0]
     plan = DispatchPlan.build(indices, E)
+    w = scores.reshape(-1)[plan.order].unsqueeze(-1)
     xs = x[plan.token]
+    if weight_input:
+        xs = (xs * w).to(gate_up.dtype)
     ys = grouped_swiglu(xs, plan.offsets, gate_up, down, act)
-    w = scores.reshape(-1)[plan.order].to(ys.dtype).unsqueeze(-1)
-    out = torch.zeros_like(x)
-    out.index_add_(0, plan.token, ys * w)
+    if not weight_input:
+        ys = ys * w.to(ys.dtype)
+    out = torch.zeros(x.shape, dtype=ys.dtype, device=x.device)
+    out.index_add_(0, plan.token, ys)
     return out
+
+
+def routed_experts(x: torch.Tensor, logits: torch.Tensor, gate_up, down, top_k: int, *, score: str = "softmax",
+                   renorm: bool = True, weight_input: bool = False, act: str = "silu") -> torch.Tensor:
+    """Experts behind router logits computed elsewhere (float32 ``[T, E]``): the device-resident plan on GPUs, the
+    eager one on the CPU.  ``x`` ``[T, H]``."""
+    if ops_native(x) and not (gate_up.requires_grad or down.requires_grad):
+        from ..ops import cuda as C
+        scores, idx, counts, _ = C.moe_route(logits, top_k, renorm, score)
+        return C.moe_experts(x, scores, idx, counts, gate_up, down, act, weight_input=weight_input)
+    _, scores, idx = topk_scores(logits, top_k, renorm, score)
+    return moe_experts(x, idx, scores, gate_up, down, act, weight_input)
 
 
 def _device_moe(x2, router_w, gate_up, down, top_k, act, gate_up_t=None, down_t=None):

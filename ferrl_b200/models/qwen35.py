@@ -534,7 +534,7 @@ class Qwen35CachedDecoder:
         return sum(t.numel() * t.element_size() for s in self.state for t in s)
 
     @torch.no_grad()
-    def prefill(self, ids, lens, rows=None):
+    def prefill(self, ids, lens, rows=None, at=None):
         m = self.m
         P, L = ids.shape
         rows = torch.arange(P, device=ids.device) if rows is None else rows
@@ -554,7 +554,7 @@ class Qwen35CachedDecoder:
                 st[0][rows] = ns[0].to(st[0].dtype)
                 st[1][rows] = ns[1]
         self.kv_len[rows] = lens.to(torch.int32)
-        last = h[torch.arange(P, device=ids.device), (lens - 1).long()]
+        last = h[(torch.arange(P, device=ids.device), (lens - 1).long()) if at is None else at]
         last = ops.rmsnorm(last, m.final_norm, m.spec.rms_norm_eps, True)
         return ops.lora_linear(last, m.head_weight(), None, None).float()
 

@@ -8,6 +8,8 @@ silent GPU fallback: a CUDA tensor with the native extension missing raises
 """
 from __future__ import annotations
 
+import torch
+
 from . import eager
 from .eager import (apply_rope, default_inv_freq, l2norm, llama3_inv_freq, rope_tables,
                     stable_softplus)
@@ -81,13 +83,12 @@ def _library_decode_attention(q, k_cache, v_cache, kv_len, scale):
         from flash_attn import flash_attn_with_kvcache
     except ImportError:
         return None
-    import torch
     return flash_attn_with_kvcache(q[:, None], k_cache, v_cache, cache_seqlens=kv_len.to(torch.int32),
                                    softmax_scale=scale, causal=True)[:, 0]
 
 
 def attention(q, k, v, *, scale, causal=True, window=0, q_offset=0, softmax_fp32=True, kv_len=None):
-    if _LIBRARY_BASELINE and q.is_cuda and not window and not q_offset and kv_len is None and q.dtype != __import__("torch").float32:
+    if _LIBRARY_BASELINE and q.is_cuda and not window and not q_offset and kv_len is None and q.dtype != torch.float32:
         return _library_attention(q, k, v, scale, causal)
     if _on_gpu(q):
         return _cuda().attention(q, k, v, scale=scale, causal=causal, window=window,
@@ -104,6 +105,54 @@ def decode_attention(q, k_cache, v_cache, kv_len, *, scale, window=0):
     if _on_gpu(q):
         return _cuda().decode_attention(q, k_cache, v_cache, kv_len, scale=scale, window=window)
     return eager.decode_attention(q, k_cache, v_cache, kv_len, scale=scale, window=window)
+
+
+def post_norm(x, y, weight, bias, eps, alpha=1.0, gate=None, gate_bias=None, history=None, coef=None, cast=None,
+              out=None):
+    """``eager.post_norm`` on a float32 stream; returns ``(next, next rounded to cast, r)``.  ``out`` (inference only)
+    is the buffer that receives ``r``."""
+    if _on_gpu(x):
+        return _cuda().post_norm(x, y, weight, bias, eps, alpha, gate, gate_bias, history, coef, cast, out)
+    nxt, r = eager.post_norm(x, y, weight, bias, eps, alpha, gate, gate_bias, history, coef)
+    if out is not None:
+        out.copy_(r)
+    return nxt, nxt if cast is None else nxt.to(cast), r
+
+
+def latent_prep(q, dkv, norm_w, eps, cos, sin, positions, *, dim, rank):
+    """``eager.latent_prep``; the kernel rotates ``q`` in place when no gradient is wanted."""
+    if _on_gpu(q):
+        return _cuda().latent_prep(q, dkv, norm_w, eps, cos, sin, positions, dim, rank)
+    return eager.latent_prep(q, dkv, norm_w, eps, cos, sin, positions, dim, rank)
+
+
+def latent_append(q, dkv, norm_w, eps, cos, sin, kv_len, cache, *, dim, rank):
+    """Decode form of ``latent_prep``: one token per row at position ``kv_len[b]``, whose latent row goes to slot
+    ``kv_len[b] % slots`` of ``cache`` ``[B,slots,width]``.  Returns the rotated ``q`` ``[B,H,dim+rot]``."""
+    if _on_gpu(q):
+        return _cuda().latent_append(q, dkv, norm_w, eps, cos, sin, kv_len, cache, dim, rank)
+    pos = kv_len[:, None].long()
+    q4, row = eager.latent_prep(q[:, None], dkv[:, None], norm_w, eps, cos, sin, pos, dim, rank)
+    cache[torch.arange(q.shape[0], device=q.device), kv_len.long() % cache.shape[1]] = row[:, 0]
+    return q4[:, 0]
+
+
+def latent_attention(q, kv, lat, *, dim, vdim, rank, scale, window=0, sink=None):
+    if _on_gpu(q):
+        return _cuda().latent_attention(q, kv, lat, dim=dim, vdim=vdim, rank=rank, scale=scale, window=window, sink=sink)
+    return eager.latent_attention(q, kv, lat, dim=dim, vdim=vdim, rank=rank, scale=scale, window=window, sink=sink)
+
+
+def latent_decode(q, uk_t, uv, cache, count, *, rank, scale, sink=None):
+    if _on_gpu(q):
+        return _cuda().latent_decode(q, uk_t, uv, cache, count, rank=rank, scale=scale, sink=sink)
+    return eager.latent_decode(q, uk_t, uv, cache, count, rank=rank, scale=scale, sink=sink)
+
+
+def linear_f32(x, w):
+    if _on_gpu(x):
+        return _cuda().linear_f32(x, w)
+    return eager.linear_f32(x, w)
 
 
 def swiglu(gate_up, act="silu"):

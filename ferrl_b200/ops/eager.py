@@ -48,6 +48,37 @@ def stable_softplus(x):
     return F.softplus(x)
 
 
+def layernorm(x, weight, bias, eps):
+    """Layer norm in fp32 (mean and mean squared deviation, ``eps`` inside the root), float32 result."""
+    xf = x.float()
+    d = xf - xf.mean(-1, keepdim=True)
+    y = d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + eps)
+    if weight is not None:
+        y = y * weight.float()
+    return y if bias is None else y + bias.float()
+
+
+def post_norm(x, y, weight, bias, eps, alpha: float = 1.0, gate=None, gate_bias=None, history=None, coef=None):
+    """Norm after the residual sum on a float32 stream: ``r = layernorm(alpha * x + y * sigmoid(gate + gate_bias))``.
+    ``y = None`` is a plain layer norm of ``x``; without ``gate`` the branch is added as it is.  With ``history``
+    ``[n, ..., W]`` (the earlier streams) and ``coef`` ``[n + 1]`` the stream that goes on is
+    ``sum_j coef[j] history[j] + coef[n] r``.  Returns ``(next, r)``, both float32."""
+    t = x.float()
+    if y is not None:
+        yf = y.float()
+        if gate is not None:
+            g = gate.float()
+            yf = yf * torch.sigmoid(g if gate_bias is None else g + gate_bias.float())
+        t = alpha * t + yf
+    r = layernorm(t, weight, bias, eps)
+    if history is None:
+        return r, r
+    nxt = coef[history.shape[0]].float() * r
+    for j in range(history.shape[0]):
+        nxt = nxt + coef[j].float() * history[j]
+    return nxt, r
+
+
 # ----------------------------------------------------------------- rope ----
 def rope_tables(inv_freq: torch.Tensor, max_pos: int, device=None):
     t = torch.arange(max_pos, dtype=torch.float32, device=inv_freq.device)
@@ -160,6 +191,68 @@ def decode_attention(q, k_cache, v_cache, kv_len, *, scale: float, window: int =
     return torch.einsum("bhs,bshd->bhd", p, vf).to(q.dtype)
 
 
+# ----------------------------------------------------- latent attention ----
+def latent_row_width(rank: int, rot: int) -> int:
+    """Elements of a cached latent row ``[c | rotated key part]``, padded so that rows start on 16-byte boundaries."""
+    return (rank + rot + 7) // 8 * 8
+
+
+def latent_prep(q, dkv, norm_w, eps, cos, sin, positions, dim: int, rank: int):
+    """``q`` ``[B,S,H,dim+rot]`` and the down projection ``dkv`` ``[B,S,rank+rot]`` -> ``(q with its last rot entries
+    rotated, latent rows [B,S,width])``: a row is the RMS-normed latent followed by the rotated key part that all
+    heads share."""
+    qr = torch.cat([q[..., :dim], apply_rope(q[..., dim:], cos, sin, positions)], dim=-1)
+    c = rmsnorm(dkv[..., :rank].float(), norm_w.float(), eps).to(dkv.dtype)
+    kr = apply_rope(dkv[..., None, rank:], cos, sin, positions)[..., 0, :]
+    row = torch.cat([c, kr], dim=-1)
+    return qr, F.pad(row, (0, latent_row_width(rank, kr.shape[-1]) - row.shape[-1]))
+
+
+def _sink_softmax(scores, sink):
+    """Softmax over the last axis of ``scores`` ``[B,H,...,K]`` (fp32, masked with ``-inf``); with ``sink`` ``[H]`` the
+    denominator also holds ``exp(sink_h)``."""
+    if sink is None:
+        return torch.nan_to_num(torch.softmax(scores, dim=-1))
+    s = sink.float().view(1, -1, *([1] * (scores.dim() - 2)))
+    m = torch.maximum(scores.amax(-1, keepdim=True), s)
+    e = torch.exp(scores - m)
+    return e / (e.sum(-1, keepdim=True) + torch.exp(s - m))
+
+
+def latent_attention(q, kv, lat, *, dim: int, vdim: int, rank: int, scale: float, window: int = 0, sink=None):
+    """Causal latent attention over whole sequences.  ``q`` ``[B,S,H,dim+rot]``, ``kv`` ``[B,S,H*(dim+vdim)]`` (the
+    unrotated keys of all heads, then the values of all heads), ``lat`` ``[B,S,width]`` whose entries
+    ``rank .. rank+rot`` are the shared rotated key part.  Returns ``[B,S,H*vdim]``."""
+    B, S, H, E = q.shape
+    rot = E - dim
+    kn = kv[..., :H * dim].reshape(B, S, H, dim).float()
+    v = kv[..., H * dim:].reshape(B, S, H, vdim).float()
+    kr = lat[..., rank:rank + rot].float()
+    scores = (torch.einsum("bihd,bjhd->bhij", q[..., :dim].float(), kn)
+              + torch.einsum("bihr,bjr->bhij", q[..., dim:].float(), kr)) * scale
+    i = torch.arange(S, device=q.device)
+    ok = i[None, :] <= i[:, None]
+    if window and window > 0:
+        ok &= i[:, None] - i[None, :] < window
+    p = _sink_softmax(scores.masked_fill(~ok, float("-inf")), sink)
+    return torch.einsum("bhij,bjhd->bihd", p, v).reshape(B, S, H * vdim).to(q.dtype)
+
+
+def latent_decode(q, uk_t, uv, cache, count, *, rank: int, scale: float, sink=None):
+    """One query per row against cached latent rows, with the key and value up projections absorbed: ``q``
+    ``[B,H,dim+rot]``, ``uk_t`` ``[H,rank,dim]``, ``uv`` ``[H,vdim,rank]``, ``cache`` ``[B,slots,width]`` of which the
+    first ``count[b]`` slots are occupied.  Returns ``[B,H*vdim]``."""
+    B, H, E = q.shape
+    dim = uk_t.shape[2]
+    qa = torch.einsum("bhd,hkd->bhk", q[..., :dim].float(), uk_t.float()).to(q.dtype).float()
+    c, kr = cache[..., :rank].float(), cache[..., rank:rank + E - dim].float()
+    scores = (torch.einsum("bhk,bsk->bhs", qa, c) + torch.einsum("bhr,bsr->bhs", q[..., dim:].float(), kr)) * scale
+    ok = torch.arange(cache.shape[1], device=q.device)[None, :] < count[:, None]
+    p = _sink_softmax(scores.masked_fill(~ok[:, None, :], float("-inf")), sink)
+    ctx = torch.einsum("bhs,bsk->bhk", p, c).to(q.dtype).float()
+    return torch.einsum("bhk,hvk->bhv", ctx, uv.float()).reshape(B, -1).to(q.dtype)
+
+
 # ------------------------------------------------------------ mlp / act ----
 def swiglu(gate_up: torch.Tensor, act: str = "silu"):
     """``act(gate) * up`` on a fused ``[..., 2F]`` tensor laid out ``[gate | up]``."""
@@ -184,6 +277,11 @@ def lora_linear(x, w, a_stack, b_stack, bias=None):
         t = F.linear(x, a_stack.to(x.dtype))
         y = y + F.linear(t, b_stack.to(x.dtype))
     return y
+
+
+def linear_f32(x, w):
+    """``x Wᵀ`` accumulated and returned in float32 (router logits, vocabulary logits)."""
+    return F.linear(x.float(), w.float())
 
 
 def lora_merge(w, a_stack, b_stack):

@@ -187,6 +187,58 @@ const char* decode_attn(const DecodeAttnArgs& a, cudaStream_t s);
 size_t decode_attn_workspace_bytes(int B, int Hq, int D, int n_splits);
 int decode_attn_pick_splits(int B, int Hkv, int max_len, int num_sms);
 
+// ---- latent attention (csrc/kernels/latent_attn.cu; tcgen05 prefill form in flash_tc.cu) ----
+struct LatentPrepArgs {
+  int dtype;
+  void* q; long long ld_q;                 // [n_tok, heads * (dim + rot)], rotated in place
+  const void* dkv; long long ld_dkv;       // [n_tok, rank + rot]
+  const float* norm_w; float eps;
+  const float* cos_t; const float* sin_t; int half; long long max_pos;   // [max_pos, half]; 2 * half <= rot
+  const long long* pos; long long S;       // prefill: position of token t is pos[t % S]
+  const int* kv_len; int slots;            // decode (kv_len set): position kv_len[t], row t's slot kv_len[t] % slots
+  void* out; int width;                    // prefill [n_tok, width]; decode [n_tok, slots, width]
+  long long n_tok; int heads, dim, rot, rank;
+};
+const char* latent_prep(const LatentPrepArgs& a, cudaStream_t s);
+struct LatentFwdArgs {
+  int dtype;
+  const void* q; const void* kn; const void* kr; const void* v; void* out;   // q [B,S,H,dim+rot], kn [B,S,H,dim], kr [B,S,rot], v [B,S,H,vdim]
+  long long q_bs, q_ts, kn_bs, kn_ts, kr_bs, kr_ts, v_bs, v_ts, o_bs, o_ts;  // batch / token strides; heads packed
+  int B, S, heads, dim, rot, vdim; float scale; int window;
+  const float* sink;                       // [heads] or null
+};
+const char* latent_fwd_any(const LatentFwdArgs& a, cudaStream_t s);
+bool latent_fwd_tc_supported(const LatentFwdArgs& a);
+size_t latent_fwd_tc_workspace_elems(const LatentFwdArgs& a);
+const char* latent_fwd_tc(const LatentFwdArgs& a, void* vt_ws, int* status, cudaStream_t s);
+// out[b, h * N + n] = sum_k x[b, h * xh + k] w[h, n, k]
+const char* head_gemm(int dtype, const void* x, long long ldx, int xh, const void* w, void* out, long long ldo, int B, int H,
+                      int N, int K, cudaStream_t s);
+struct LatentDecodeArgs {
+  int dtype;
+  const void* qa;                          // absorbed queries [B, heads, rank]
+  const void* qr; long long ld_qr; int qr_hs;   // rotated query parts: row stride, head stride
+  const void* cache; int slots, width;     // [B, slots, width]: latent, rotated key part
+  const int* count;                        // occupied slots per row
+  const float* sink; void* ctx; float* ws; // ctx [B, heads, rank]; ws B * heads * n_splits * (rank + 2) floats
+  int B, heads, rank, rot; float scale;
+};
+bool latent_decode_tc_supported(const LatentDecodeArgs& a);
+int latent_decode_splits(const LatentDecodeArgs& a, int num_sms);
+const char* latent_decode(const LatentDecodeArgs& a, int n_splits, cudaStream_t s);
+
+// ---- residual sum + layer norm + depth average (csrc/kernels/post_norm.cu) ----
+struct PostNormArgs {
+  const float* x; long long rows; int W;
+  const void* y; long long ld_y; int y_dtype;            // branch output or null
+  const void* gate; long long ld_gate; int gate_dtype;   // gate logits or null
+  const float* gate_bias; const float* w; const float* b;
+  float eps, alpha;
+  const float* history; long long hist_stride; int n_hist; const float* coef;   // coef [n_hist + 1] or null
+  float* r; float* next; void* cast; int cast_dtype;     // outputs, each may be null
+};
+const char* post_norm(const PostNormArgs& a, cudaStream_t s);
+
 // ---- flash attention (prefill / training) ----
 struct FlashArgs {
   const void* q; const void* k; const void* v; void* o; float* lse;   // bf16; lse [B,Hq,Sq]
@@ -222,8 +274,16 @@ const char* sample_rows(int dtype, const void* logits, long long ld, const long 
                         int rows, int V, float temperature, float top_p, cudaStream_t s);
 
 // ---- mixture of experts (csrc/moe/moe.cu); all return nullptr on success
-const char* moe_route(const float* logits, long long ld, int T, int E, int k, bool renorm, float* probs, float* scores,
+// score: 0 softmax over the experts, 1 sigmoid of each logit
+const char* moe_route(const float* logits, long long ld, int T, int E, int k, bool renorm, int score, float* probs, float* scores,
                       int* idx, int* counts, cudaStream_t stream);
+// any type and size: the gather, grouped product and combine of the same plan without tensor cores
+const char* moe_gather_any(int dtype, const void* x, long long ldx, const int* token_of, const float* pair_w, const int* row_of,
+                           int n_pairs, float* row_scale, int rows, int H, void* xs, cudaStream_t stream);
+const char* moe_grouped_any(int dtype, const void* xs, const void* W, const int* tile_expert, int rows, int N, int K, void* out,
+                            cudaStream_t stream);
+const char* moe_combine_any(int dtype, const void* ys, const int* row_of, const float* w, int T, int k, int H, void* out,
+                            cudaStream_t stream);
 const char* moe_plan(const int* idx, const int* counts, int n_pairs, int k, int E, int max_rows, int* row_of,
                      int* token_of, int* tile_expert, int* seg_start, cudaStream_t stream);
 const char* moe_gather(const void* x, long long ldx, const int* token_of, const float* pair_w, const int* row_of,

@@ -644,9 +644,13 @@ std::tuple<Tensor, Tensor> gdn_chunk_fwd(const Tensor& q, const Tensor& k, const
   return {out, S};
 }
 
+Tensor glu_fwd(const Tensor& gu, int64_t act);
+
 // ---------------------------------------------------------------- mixture of experts
 // logits [T, E] fp32 -> (probs [T,E] f32, scores [T,k] f32, idx [T,k] i32, counts [E] i32)
-std::tuple<Tensor, Tensor, Tensor, Tensor> moe_route(const Tensor& logits, int64_t k, bool renorm) {
+// score: 0 softmax over the experts, 1 sigmoid of each logit
+std::tuple<Tensor, Tensor, Tensor, Tensor> moe_route(const Tensor& logits, int64_t k, bool renorm, int64_t score) {
+  TORCH_CHECK(score == 0 || score == 1, "moe_route: score 0 (softmax) or 1 (sigmoid)");
   TORCH_CHECK(logits.is_cuda() && logits.scalar_type() == at::kFloat && logits.dim() == 2 && logits.stride(1) == 1, "moe_route: fp32 [T,E]");
   c10::cuda::CUDAGuard guard(logits.device());
   const int64_t T = logits.size(0), E = logits.size(1);
@@ -654,7 +658,7 @@ std::tuple<Tensor, Tensor, Tensor, Tensor> moe_route(const Tensor& logits, int64
   Tensor scores = out_empty({T, k}, logits.options());
   Tensor idx = out_empty({T, k}, logits.options().dtype(at::kInt));
   Tensor counts = out_empty({E}, logits.options().dtype(at::kInt));
-  FERRL_CHECK(ferrl::moe_route(logits.data_ptr<float>(), logits.stride(0), T, E, k, renorm, probs.data_ptr<float>(),
+  FERRL_CHECK(ferrl::moe_route(logits.data_ptr<float>(), logits.stride(0), T, E, k, renorm, static_cast<int>(score), probs.data_ptr<float>(),
                                scores.data_ptr<float>(), idx.data_ptr<int>(), counts.data_ptr<int>(), stream()));
   return {probs, scores, idx, counts};
 }
@@ -718,6 +722,35 @@ Tensor moe_grouped_gemm(const Tensor& xs, const Tensor& W, const Tensor& tile_ex
   a.status = status_word(); a.num_sms = num_sms();
   a.force_bn = a.N >= 256 ? 256 : (a.N >= 128 ? 128 : 64);
   FERRL_CHECK(ferrl::gemm_bf16(a, stream()));
+  return out;
+}
+
+// The routed experts of one plan at any size and type (fp32, or bf16 sizes the tensor-core path does not take):
+// out = sum over a token's experts of down(act(gate) * up); `w` multiplies inputs (weight_input) or outputs.
+Tensor moe_experts_any(const Tensor& x, const Tensor& w, const Tensor& idx, const Tensor& counts, const Tensor& gate_up, const Tensor& down,
+                       int64_t act, bool weight_input) {
+  TORCH_CHECK(x.is_cuda() && x.dim() == 2 && x.stride(1) == 1 && gate_up.dim() == 3 && down.dim() == 3 && gate_up.is_contiguous() &&
+                  down.is_contiguous() && gate_up.scalar_type() == x.scalar_type() && down.scalar_type() == x.scalar_type() &&
+                  gate_up.size(2) == x.size(1) && down.size(1) == x.size(1) && gate_up.size(1) == 2 * down.size(2) &&
+                  gate_up.size(0) == counts.numel() && down.size(0) == counts.numel(),
+              "moe_experts_any: x [T,H], gate_up [E,2I,H], down [E,H,I] of one type");
+  TORCH_CHECK(w.scalar_type() == at::kFloat && w.is_contiguous() && w.numel() == idx.numel() && idx.size(0) == x.size(0), "moe_experts_any: weights f32 [T,k]");
+  c10::cuda::CUDAGuard guard(x.device());
+  auto plan = moe_plan(idx, counts);
+  const Tensor &row_of = std::get<0>(plan), &token_of = std::get<1>(plan), &tile_expert = std::get<2>(plan);
+  const int64_t rows = token_of.size(0), H = x.size(1), I = down.size(2), T = x.size(0), k = idx.size(1);
+  Tensor xs = out_empty({rows, H}, x.options());
+  Tensor row_scale = out_zeros({rows}, x.options().dtype(at::kFloat));
+  FERRL_CHECK(ferrl::moe_gather_any(dt(x), x.data_ptr(), x.stride(0), token_of.data_ptr<int>(), weight_input ? w.data_ptr<float>() : nullptr,
+                                    row_of.data_ptr<int>(), row_of.numel(), row_scale.data_ptr<float>(), rows, H, xs.data_ptr(), stream()));
+  Tensor gu = out_zeros({rows, 2 * I}, x.options());
+  FERRL_CHECK(ferrl::moe_grouped_any(dt(x), xs.data_ptr(), gate_up.data_ptr(), tile_expert.data_ptr<int>(), rows, 2 * I, H, gu.data_ptr(), stream()));
+  Tensor mid = glu_fwd(gu, act);
+  Tensor ys = out_zeros({rows, H}, x.options());
+  FERRL_CHECK(ferrl::moe_grouped_any(dt(x), mid.data_ptr(), down.data_ptr(), tile_expert.data_ptr<int>(), rows, H, I, ys.data_ptr(), stream()));
+  Tensor out = out_empty({T, H}, x.options());
+  FERRL_CHECK(ferrl::moe_combine_any(dt(x), ys.data_ptr(), row_of.data_ptr<int>(), weight_input ? nullptr : w.data_ptr<float>(), T, k, H,
+                                     out.data_ptr(), stream()));
   return out;
 }
 
@@ -1094,6 +1127,193 @@ Tensor decode_attn(const Tensor& q, const Tensor& kc, const Tensor& vc, const Te
   return out;
 }
 
+// ---------------------------------------------------------------- latent attention
+static void f32_vec(const Tensor& t, int64_t n, const char* what) {
+  TORCH_CHECK(t.is_cuda() && t.scalar_type() == at::kFloat && t.is_contiguous() && t.numel() == n, what);
+}
+static void fill_latent_prep(ferrl::LatentPrepArgs& a, const Tensor& q, const Tensor& dkv, const Tensor& norm_w, double eps, const Tensor& cos_t,
+                             const Tensor& sin_t, int64_t dim, int64_t rank) {
+  // q [n_tok, H, dim + rot] and dkv [n_tok, rank + rot]: views into the fused projection are fine
+  TORCH_CHECK(q.is_cuda() && q.dim() == 3 && q.stride(2) == 1 && q.stride(1) == q.size(2) && dkv.dim() == 2 && dkv.stride(1) == 1 &&
+                  dkv.size(0) == q.size(0) && dkv.scalar_type() == q.scalar_type(), "latent_prep: q [n,H,dim+rot], dkv [n,rank+rot]");
+  a.dtype = dt(q);
+  a.n_tok = q.size(0); a.heads = q.size(1); a.dim = dim; a.rot = q.size(2) - dim; a.rank = rank;
+  TORCH_CHECK(a.rot > 0 && dkv.size(1) == rank + a.rot, "latent_prep: sizes");
+  f32_vec(norm_w, rank, "latent_prep: norm weight f32 [rank]");
+  TORCH_CHECK(cos_t.scalar_type() == at::kFloat && cos_t.is_contiguous() && cos_t.dim() == 2 && cos_t.size(0) > 0 &&
+                  sin_t.scalar_type() == at::kFloat && sin_t.is_contiguous() && sin_t.sizes() == cos_t.sizes() &&
+                  2 * cos_t.size(1) <= a.rot, "latent_prep: tables f32 [max_pos, half]");
+  a.q = q.data_ptr(); a.ld_q = q.stride(0); a.dkv = dkv.data_ptr(); a.ld_dkv = dkv.stride(0);
+  a.norm_w = norm_w.data_ptr<float>(); a.eps = static_cast<float>(eps);
+  a.cos_t = cos_t.data_ptr<float>(); a.sin_t = sin_t.data_ptr<float>(); a.half = cos_t.size(1); a.max_pos = cos_t.size(0);
+}
+
+// whole sequences: token t of the flattened [B, S] batch is at position pos[t % S]; returns the rows [n_tok, width]
+Tensor latent_prep(Tensor q, const Tensor& dkv, const Tensor& norm_w, double eps, const Tensor& cos_t, const Tensor& sin_t, const Tensor& pos,
+                   int64_t dim, int64_t rank, int64_t width) {
+  c10::cuda::CUDAGuard guard(q.device());
+  ferrl::LatentPrepArgs a{};
+  fill_latent_prep(a, q, dkv, norm_w, eps, cos_t, sin_t, dim, rank);
+  TORCH_CHECK(pos.is_cuda() && pos.scalar_type() == at::kLong && pos.is_contiguous() && pos.numel() > 0, "latent_prep: positions int64");
+  TORCH_CHECK(width >= rank + a.rot, "latent_prep: row width");
+  Tensor out = out_empty({a.n_tok, width}, q.options());
+  a.pos = reinterpret_cast<const long long*>(pos.data_ptr<int64_t>()); a.S = pos.numel();
+  a.out = out.data_ptr(); a.width = width;
+  FERRL_CHECK(ferrl::latent_prep(a, stream()));
+  return out;
+}
+
+// one token per row: position kv_len[b], row b's slot kv_len[b] % slots of cache [B, slots, width]
+void latent_append(Tensor q, const Tensor& dkv, const Tensor& norm_w, double eps, const Tensor& cos_t, const Tensor& sin_t, const Tensor& kv_len,
+                   Tensor cache, int64_t dim, int64_t rank) {
+  c10::cuda::CUDAGuard guard(q.device());
+  ferrl::LatentPrepArgs a{};
+  fill_latent_prep(a, q, dkv, norm_w, eps, cos_t, sin_t, dim, rank);
+  TORCH_CHECK(kv_len.is_cuda() && kv_len.scalar_type() == at::kInt && kv_len.is_contiguous() && kv_len.numel() == a.n_tok, "latent_append: kv_len int32 [B]");
+  TORCH_CHECK(cache.is_cuda() && cache.dim() == 3 && cache.is_contiguous() && cache.scalar_type() == q.scalar_type() && cache.size(0) == a.n_tok &&
+                  cache.size(1) > 0 && cache.size(2) >= rank + a.rot, "latent_append: cache [B, slots, width]");
+  a.kv_len = kv_len.data_ptr<int>(); a.slots = cache.size(1); a.out = cache.data_ptr(); a.width = cache.size(2);
+  FERRL_CHECK(ferrl::latent_prep(a, stream()));
+}
+
+// q [B,S,H,dim+rot], kv [B,S,H*(dim+vdim)], lat [B,S,width] -> [B,S,H*vdim]; variant 1 forces the any-size kernel
+Tensor latent_fwd(const Tensor& q, const Tensor& kv, const Tensor& lat, int64_t dim, int64_t vdim, int64_t rank, double scale, int64_t window,
+                  const optional<Tensor>& sink, int64_t variant) {
+  TORCH_CHECK(q.is_cuda() && q.dim() == 4 && q.stride(3) == 1 && q.stride(2) == q.size(3) && kv.dim() == 3 && kv.stride(2) == 1 &&
+                  lat.dim() == 3 && lat.stride(2) == 1 && kv.scalar_type() == q.scalar_type() && lat.scalar_type() == q.scalar_type(),
+              "latent_fwd: q [B,S,H,dim+rot], kv [B,S,H*(dim+vdim)], lat [B,S,width]");
+  c10::cuda::CUDAGuard guard(q.device());
+  ferrl::LatentFwdArgs a{};
+  a.dtype = dt(q);
+  a.B = q.size(0); a.S = q.size(1); a.heads = q.size(2); a.dim = dim; a.rot = q.size(3) - dim; a.vdim = vdim;
+  TORCH_CHECK(a.rot > 0 && dim > 0 && vdim > 0 && kv.size(0) == a.B && kv.size(1) == a.S && kv.size(2) == a.heads * (dim + vdim) &&
+                  lat.size(0) == a.B && lat.size(1) == a.S && lat.size(2) >= rank + a.rot && window >= 0, "latent_fwd: sizes");
+  const int64_t es = q.element_size();
+  a.q = q.data_ptr(); a.kn = kv.data_ptr();
+  a.kr = static_cast<const char*>(lat.data_ptr()) + rank * es;
+  a.v = static_cast<const char*>(kv.data_ptr()) + a.heads * dim * es;
+  // a size-1 dimension has an arbitrary stride
+  auto ts = [&](const Tensor& t) { return a.S > 1 ? t.stride(1) : (a.B > 1 ? t.stride(0) : (t.size(-1) + 7) / 8 * 8); };
+  auto bs = [&](const Tensor& t) { return a.B > 1 ? t.stride(0) : ts(t) * a.S; };
+  a.q_ts = a.S > 1 || a.B > 1 ? ts(q) : (q.size(2) * q.size(3) + 7) / 8 * 8;
+  a.q_bs = a.B > 1 ? q.stride(0) : a.q_ts * a.S;
+  a.kn_bs = a.v_bs = bs(kv); a.kn_ts = a.v_ts = ts(kv); a.kr_bs = bs(lat); a.kr_ts = ts(lat);
+  a.scale = scale; a.window = window;
+  if (sink.has_value() && sink->defined()) {
+    f32_vec(*sink, a.heads, "latent_fwd: sink f32 [H]");
+    a.sink = sink->data_ptr<float>();
+  }
+  Tensor out = out_empty({a.B, a.S, a.heads * vdim}, q.options());
+  a.out = out.data_ptr(); a.o_ts = a.heads * vdim; a.o_bs = a.o_ts * a.S;
+  if (variant == 0 && ferrl::latent_fwd_tc_supported(a)) {
+    Tensor vt = out_empty({static_cast<long long>(ferrl::latent_fwd_tc_workspace_elems(a))}, q.options());
+    FERRL_CHECK(ferrl::latent_fwd_tc(a, vt.data_ptr(), status_word(), stream()));
+    return out;
+  }
+  FERRL_CHECK(ferrl::latent_fwd_any(a, stream()));
+  return out;
+}
+
+// q [B,H,dim+rot] (rotated), uk_t [H,rank,dim], uv [H,vdim,rank], cache [B,slots,width], count i32 [B] -> [B, H*vdim]
+Tensor latent_decode(const Tensor& q, const Tensor& uk_t, const Tensor& uv, const Tensor& cache, const Tensor& count, double scale,
+                     const optional<Tensor>& sink, int64_t splits) {
+  TORCH_CHECK(q.is_cuda() && q.dim() == 3 && q.stride(2) == 1 && q.stride(1) == q.size(2) && uk_t.dim() == 3 && uk_t.is_contiguous() &&
+                  uv.dim() == 3 && uv.is_contiguous() && cache.dim() == 3 && cache.is_contiguous() && uk_t.scalar_type() == q.scalar_type() &&
+                  uv.scalar_type() == q.scalar_type() && cache.scalar_type() == q.scalar_type(), "latent_decode: layout");
+  c10::cuda::CUDAGuard guard(q.device());
+  ferrl::LatentDecodeArgs a{};
+  a.dtype = dt(q);
+  a.B = q.size(0); a.heads = q.size(1); a.rank = uk_t.size(1);
+  const int64_t dim = uk_t.size(2), vdim = uv.size(1);
+  a.rot = q.size(2) - dim;
+  TORCH_CHECK(a.rot > 0 && uk_t.size(0) == a.heads && uv.size(0) == a.heads && uv.size(2) == a.rank && cache.size(0) == a.B &&
+                  cache.size(2) >= a.rank + a.rot, "latent_decode: sizes");
+  TORCH_CHECK(count.is_cuda() && count.scalar_type() == at::kInt && count.is_contiguous() && count.numel() == a.B, "latent_decode: count int32 [B]");
+  if (sink.has_value() && sink->defined()) {
+    f32_vec(*sink, a.heads, "latent_decode: sink f32 [H]");
+    a.sink = sink->data_ptr<float>();
+  }
+  Tensor qa = out_empty({a.B, a.heads, a.rank}, q.options());
+  FERRL_CHECK(ferrl::head_gemm(a.dtype, q.data_ptr(), q.stride(0), q.size(2), uk_t.data_ptr(), qa.data_ptr(),
+                               static_cast<long long>(a.heads) * a.rank, a.B, a.heads, a.rank, dim, stream()));
+  Tensor ctx = out_empty({a.B, a.heads, a.rank}, q.options());
+  a.qa = qa.data_ptr();
+  a.qr = static_cast<const char*>(q.data_ptr()) + dim * q.element_size();
+  a.ld_qr = q.stride(0); a.qr_hs = q.size(2);
+  a.cache = cache.data_ptr(); a.slots = cache.size(1); a.width = cache.size(2); a.count = count.data_ptr<int>();
+  a.ctx = ctx.data_ptr(); a.scale = scale;
+  int n = 1;
+  Tensor ws;
+  if (ferrl::latent_decode_tc_supported(a)) {
+    n = splits > 0 ? static_cast<int>(splits) : ferrl::latent_decode_splits(a, num_sms());
+    if (n > 1) {
+      ws = out_empty({static_cast<long long>(a.B) * a.heads * n * (a.rank + 2)}, q.options().dtype(at::kFloat));
+      a.ws = ws.data_ptr<float>();
+    }
+  }
+  FERRL_CHECK(ferrl::latent_decode(a, n, stream()));
+  Tensor out = out_empty({a.B, a.heads * vdim}, q.options());
+  FERRL_CHECK(ferrl::head_gemm(a.dtype, ctx.data_ptr(), static_cast<long long>(a.heads) * a.rank, a.rank, uv.data_ptr(), out.data_ptr(),
+                               a.heads * vdim, a.B, a.heads, vdim, a.rank, stream()));
+  return out;
+}
+
+// see csrc/kernels/post_norm.cu; returns (next f32, next in the compute dtype (next itself for f32), r f32)
+std::tuple<Tensor, Tensor, Tensor> post_norm(const Tensor& x, const optional<Tensor>& y, const optional<Tensor>& gate, const optional<Tensor>& gate_bias,
+                                             const Tensor& w, const optional<Tensor>& b, double eps, double alpha, const optional<Tensor>& history,
+                                             const optional<Tensor>& coef, bool cast_bf16, const optional<Tensor>& r_out) {
+  TORCH_CHECK(x.is_cuda() && x.scalar_type() == at::kFloat && x.is_contiguous() && x.dim() >= 1 && x.size(-1) > 0, "post_norm: x f32");
+  c10::cuda::CUDAGuard guard(x.device());
+  auto has = [](const optional<Tensor>& t) { return t.has_value() && t->defined(); };
+  ferrl::PostNormArgs a{};
+  const int64_t W = x.size(-1), rows = x.numel() / W;
+  a.x = x.data_ptr<float>(); a.rows = rows; a.W = W; a.eps = eps; a.alpha = alpha;
+  a.cast_dtype = cast_bf16 ? ferrl::kBF16 : ferrl::kF32;
+  a.y_dtype = a.gate_dtype = a.cast_dtype;
+  if (has(y)) {
+    TORCH_CHECK(y->is_cuda() && y->dim() == 2 && y->size(0) == rows && y->size(1) == W && y->stride(1) == 1, "post_norm: y [rows, W]");
+    a.y = y->data_ptr(); a.ld_y = y->stride(0); a.y_dtype = dt(*y);
+  }
+  if (has(gate)) {
+    TORCH_CHECK(gate->is_cuda() && has(y) && gate->dim() == 2 && gate->size(0) == rows && gate->size(1) == W && gate->stride(1) == 1, "post_norm: gate [rows, W]");
+    a.gate = gate->data_ptr(); a.ld_gate = gate->stride(0); a.gate_dtype = dt(*gate);
+    if (has(gate_bias)) {
+      f32_vec(*gate_bias, W, "post_norm: gate bias f32 [W]");
+      a.gate_bias = gate_bias->data_ptr<float>();
+    }
+  }
+  f32_vec(w, W, "post_norm: weight f32 [W]");
+  a.w = w.data_ptr<float>();
+  if (has(b)) {
+    f32_vec(*b, W, "post_norm: bias f32 [W]");
+    a.b = b->data_ptr<float>();
+  }
+  Tensor next = out_empty(x.sizes(), x.options()), r = next;
+  if (has(r_out)) {
+    f32_vec(*r_out, x.numel(), "post_norm: result buffer");
+    r = *r_out;
+    a.r = r.data_ptr<float>();
+  }
+  if (has(history)) {
+    TORCH_CHECK(has(coef) && history->is_cuda() && history->scalar_type() == at::kFloat && history->is_contiguous() &&
+                    history->numel() == history->size(0) * x.numel(), "post_norm: history f32 [n, ...] with coefficients");
+    f32_vec(*coef, history->size(0) + 1, "post_norm: coefficients f32 [n + 1]");
+    a.history = history->data_ptr<float>(); a.hist_stride = x.numel(); a.n_hist = history->size(0); a.coef = coef->data_ptr<float>();
+    if (!a.r) {
+      r = out_empty(x.sizes(), x.options());
+      a.r = r.data_ptr<float>();
+    }
+  }
+  a.next = next.data_ptr<float>();
+  Tensor cast = next;
+  if (cast_bf16) {
+    cast = out_empty(x.sizes(), x.options().dtype(at::kBFloat16));
+    a.cast = cast.data_ptr();
+  }
+  FERRL_CHECK(ferrl::post_norm(a, stream()));
+  return {next, cast, r};
+}
+
 void fill_flash(ferrl::FlashArgs& a, const Tensor& q, const Tensor& k, const Tensor& v, double scale, bool causal,
                 int64_t window, int64_t q_offset) {
   TORCH_CHECK(q.is_cuda() && q.scalar_type() == at::kBFloat16 && k.scalar_type() == at::kBFloat16 &&
@@ -1412,7 +1632,7 @@ TORCH_LIBRARY(ferrl_b200, m) {
   m.def("gdn_tc_bwd(Tensor q, Tensor k, Tensor v, Tensor beta, Tensor Gc, Tensor gl, Tensor Tm, Tensor Wn, Tensor Kd, Tensor Vn, Tensor Sin, Tensor dO, Tensor? dS_final) -> Tensor[]", &gdn_tc_bwd);
   m.def("gdn_decode_step_raw(Tensor q, Tensor k, Tensor v, Tensor a, Tensor b, Tensor A_log, Tensor dt_bias, Tensor(a!) S, bool l2norm, float eps) -> Tensor", &gdn_decode_step_raw);
   m.def("gdn_decode_step(Tensor q, Tensor k, Tensor v, Tensor g, Tensor beta, Tensor(a!) S, bool l2norm, float eps) -> Tensor", &gdn_decode_step);
-  m.def("moe_route(Tensor logits, int k, bool renorm) -> (Tensor, Tensor, Tensor, Tensor)", &moe_route);
+  m.def("moe_route(Tensor logits, int k, bool renorm, int score=0) -> (Tensor, Tensor, Tensor, Tensor)", &moe_route);
   m.def("moe_plan(Tensor idx, Tensor counts) -> (Tensor, Tensor, Tensor, Tensor)", &moe_plan);
   m.def("moe_gather(Tensor x, Tensor token_of, Tensor? pair_w, Tensor row_of) -> Tensor", &moe_gather);
   m.def("moe_grouped_gemm(Tensor xs, Tensor W, Tensor tile_expert, Tensor(a!)? out=None) -> Tensor(a!)", &moe_grouped_gemm);
@@ -1436,6 +1656,12 @@ TORCH_LIBRARY(ferrl_b200, m) {
   m.def("grpo_loss_rows(Tensor logp, Tensor logp_old, Tensor? logp_ref, Tensor adv, Tensor mask, Tensor? tis, float eps_lo, float eps_hi, float beta, bool seq_level, bool want_grad) -> (Tensor, Tensor, Tensor)", &grpo_loss_rows);
   m.def("grpo_scale_rows(Tensor(a!) dlogp, Tensor row_scale) -> ()", &grpo_scale_rows);
   m.def("decode_attn(Tensor q, Tensor kc, Tensor vc, Tensor kv_len, float scale, int window, int n_splits, Tensor? block_table, int page, int variant=0, Tensor? prefix_len=None, int group=1, int prefix_splits=1) -> Tensor", &decode_attn);
+  m.def("latent_prep(Tensor(a!) q, Tensor dkv, Tensor norm_w, float eps, Tensor cos_t, Tensor sin_t, Tensor pos, int dim, int rank, int width) -> Tensor", &latent_prep);
+  m.def("latent_append(Tensor(a!) q, Tensor dkv, Tensor norm_w, float eps, Tensor cos_t, Tensor sin_t, Tensor kv_len, Tensor(b!) cache, int dim, int rank) -> ()", &latent_append);
+  m.def("latent_fwd(Tensor q, Tensor kv, Tensor lat, int dim, int vdim, int rank, float scale, int window, Tensor? sink, int variant=0) -> Tensor", &latent_fwd);
+  m.def("latent_decode(Tensor q, Tensor uk_t, Tensor uv, Tensor cache, Tensor count, float scale, Tensor? sink, int splits=0) -> Tensor", &latent_decode);
+  m.def("post_norm(Tensor x, Tensor? y, Tensor? gate, Tensor? gate_bias, Tensor w, Tensor? b, float eps, float alpha, Tensor? history, Tensor? coef, bool cast_bf16, Tensor? r_out) -> (Tensor, Tensor, Tensor)", &post_norm);
+  m.def("moe_experts_any(Tensor x, Tensor w, Tensor idx, Tensor counts, Tensor gate_up, Tensor down, int act, bool weight_input) -> Tensor", &moe_experts_any);
   m.def("gemm_norm(Tensor A, Tensor B, Tensor? residual, Tensor? ss_in, float eps, int glu_act, bool want_ss, bool static_b=True) -> (Tensor, Tensor)", &gemm_norm);
   m.def("row_sumsq(Tensor x) -> Tensor", &row_sumsq);
   m.def("gemm_glu(Tensor A, Tensor B, int act, bool static_b=False) -> Tensor", &gemm_glu);

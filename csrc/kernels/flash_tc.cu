@@ -654,22 +654,35 @@ __global__ void transpose_v_hd_kernel(const __nv_bfloat16* __restrict__ v, long 
   }
 }
 
-template <int HD, int KT>
+// Score width and value width are template parameters of their own: NQ 64-column atoms of query / key and HD value
+// columns.  The latent form (LAT) assembles a score operand from two parts: the atoms of the unrotated entries of a
+// head, then those of the rotated ones, which all heads share on the key side.  Each part is zero-filled up to whole
+// atoms by its tensor map, and `kmask` names the 16-column steps that hold anything.
+struct LatentTcParams {
+  int na0;                  // atoms of the unrotated part
+  uint32_t kmask;           // bit ks: MMA step ks (16 columns) is not all padding
+  int vdim;                 // stored value columns per head (<= HD)
+  const float* sink;        // [heads] or null: exp(sink) joins the softmax denominator
+};
+
+template <int NQ, int HD, int KT>
 struct Tc3Cfg {
-  static constexpr int Q_BYTES = FT * HD * 2;          // HD/64 atoms of [128 rows x 64 cols]
+  static constexpr int Q_BYTES = NQ * ATOM;            // NQ atoms of [128 rows x 64 cols]
   static constexpr int K_ATOM = KT * 128;              // [KT keys x 64 dims]
-  static constexpr int K_BYTES = (HD / 64) * K_ATOM;
+  static constexpr int K_BYTES = NQ * K_ATOM;
   static constexpr int V_ATOM = HD * 128;              // [HD dims x 64 keys]
   static constexpr int V_BYTES = (KT / 64) * V_ATOM;
   static constexpr int SMEM = Q_BYTES + 2 * K_BYTES + 2 * V_BYTES + 1024 + 256;
   static_assert(3 * KT + HD <= 512, "tensor memory columns");
+  static_assert(SMEM <= 227 * 1024, "shared memory");
 };
 
-template <int HD, int KT>
+template <int NQ, int HD, int KT, bool LAT>
 __global__ void __launch_bounds__(192, 1)
 flash_fwd_tc3_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                     const __grid_constant__ CUtensorMap tmVt, FlashTcParams p, int window) {
-  using C = Tc3Cfg<HD, KT>;
+                     const __grid_constant__ CUtensorMap tmVt, const __grid_constant__ CUtensorMap tmQr,
+                     const __grid_constant__ CUtensorMap tmKr, FlashTcParams p, int window, LatentTcParams lt) {
+  using C = Tc3Cfg<NQ, HD, KT>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;
@@ -730,15 +743,29 @@ flash_fwd_tc3_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       // ------------------------------------------------------------------ TMA producer
       mbar_expect_tx(q_full, C::Q_BYTES);
 #pragma unroll
-      for (int a = 0; a < HD / 64; ++a) tma_load_2d(sQ + a * ATOM, &tmQ, q_full, hq * HD + a * 64, b * p.S + q0);
+      for (int a = 0; a < NQ; ++a) {
+        if constexpr (LAT) {
+          if (a < lt.na0) tma_load_3d(sQ + a * ATOM, &tmQ, q_full, a * 64, hq, b * p.S + q0);
+          else tma_load_3d(sQ + a * ATOM, &tmQr, q_full, (a - lt.na0) * 64, hq, b * p.S + q0);
+        } else {
+          tma_load_2d(sQ + a * ATOM, &tmQ, q_full, hq * HD + a * 64, b * p.S + q0);
+        }
+      }
       for (int jj = 0; jj < n_kv; ++jj) {
         const int j = j_lo + jj, st = jj & 1;
         const uint32_t ph = (jj >> 1) & 1;
         if (!mbar_wait(&k_empty[st], ph ^ 1, abort_flag, p.status, kStatusWaitTimeoutProducer)) break;
         mbar_expect_tx(&k_full[st], C::K_BYTES);
 #pragma unroll
-        for (int a = 0; a < HD / 64; ++a)
-          tma_load_2d(sK + st * C::K_BYTES + a * C::K_ATOM, &tmK, &k_full[st], hk * HD + a * 64, b * p.S + j * KT);
+        for (int a = 0; a < NQ; ++a) {
+          uint8_t* dst = sK + st * C::K_BYTES + a * C::K_ATOM;
+          if constexpr (LAT) {
+            if (a < lt.na0) tma_load_3d(dst, &tmK, &k_full[st], a * 64, hk, b * p.S + j * KT);
+            else tma_load_2d(dst, &tmKr, &k_full[st], (a - lt.na0) * 64, b * p.S + j * KT);
+          } else {
+            tma_load_2d(dst, &tmK, &k_full[st], hk * HD + a * 64, b * p.S + j * KT);
+          }
+        }
         if (!mbar_wait(&v_empty[st], ph ^ 1, abort_flag, p.status, kStatusWaitTimeoutProducer)) break;
         mbar_expect_tx(&v_full[st], C::V_BYTES);
 #pragma unroll
@@ -763,8 +790,8 @@ flash_fwd_tc3_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       const uint32_t ts = st ? tS1 : tS0;
       if (elect_one()) {
 #pragma unroll
-        for (int ks = 0; ks < HD / 16; ++ks)
-          umma(ts, desc_adv(dq, (ks >> 2) * ATOM + (ks & 3) * 32), desc_adv(dk, (ks >> 2) * C::K_ATOM + (ks & 3) * 32), idesc_qk,
+        for (int ks = 0; ks < NQ * 4; ++ks)
+          if (!LAT || ((lt.kmask >> ks) & 1u)) umma(ts, desc_adv(dq, (ks >> 2) * ATOM + (ks & 3) * 32), desc_adv(dk, (ks >> 2) * C::K_ATOM + (ks & 3) * 32), idesc_qk,
                ks > 0 ? 1u : 0u);
         umma_commit(&s_full[st]);
         umma_commit(&k_empty[st]);
@@ -895,8 +922,11 @@ flash_fwd_tc3_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       ok = false;
     tc_fence_after();
     if (ok) {      // warp-uniform: the TMEM loads are warp-collective, only the stores are per row
+      if constexpr (LAT) {
+        if (lt.sink && row < p.S) l_run += exp2f(lt.sink[hq] * kLog2e - m_used * c);   // a row of the sequence sees itself
+      }
       const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-      __nv_bfloat16* orow = p.out + b * p.o_bs + static_cast<long long>(row) * p.o_ts + hq * HD;
+      __nv_bfloat16* orow = p.out + b * p.o_bs + static_cast<long long>(row) * p.o_ts + hq * (LAT ? lt.vdim : HD);
 #pragma unroll 1
       for (int cc = 0; cc < HD; cc += 32) {
         uint32_t ov[32];
@@ -906,6 +936,7 @@ flash_fwd_tc3_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         if (row < p.S) {
 #pragma unroll
           for (int ch = 0; ch < 4; ++ch) {
+            if (LAT && cc + ch * 8 >= lt.vdim) break;
             uint4 w;
             __nv_bfloat162* wh = reinterpret_cast<__nv_bfloat162*>(&w);
 #pragma unroll
@@ -930,7 +961,7 @@ flash_fwd_tc3_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
 
 template <int HD, int KT>
 const char* launch_tc3(const FlashArgs& a, void* vt_ws, int* status, cudaStream_t stream) {
-  using C = Tc3Cfg<HD, KT>;
+  using C = Tc3Cfg<HD / 64, HD, KT>;
   const int s_pad = (a.Sk + 63) / 64 * 64;
   constexpr int tsm = 64 * (HD + 2) * 2;
   transpose_v_hd_kernel<HD><<<dim3(s_pad / 64, a.Hkv, a.B), 256, tsm, stream>>>(static_cast<const __nv_bfloat16*>(a.v), a.v_bs, a.v_ts,
@@ -946,16 +977,109 @@ const char* launch_tc3(const FlashArgs& a, void* vt_ws, int* status, cudaStream_
   FlashTcParams p{};
   p.out = static_cast<__nv_bfloat16*>(a.o); p.o_bs = a.o_bs; p.o_ts = a.o_ts; p.lse = a.lse;
   p.B = a.B; p.S = a.Sq; p.Hq = a.Hq; p.Hkv = a.Hkv; p.scale = a.scale; p.status = status;
-  auto kern = flash_fwd_tc3_kernel<HD, KT>;
+  auto kern = flash_fwd_tc3_kernel<HD / 64, HD, KT, false>;
   if (!FERRL_ONCE_PER_DEVICE(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM) == cudaSuccess))
     return "flash_fwd_tc: cannot reserve shared memory";
   dim3 grid((a.Sq + FT - 1) / FT, a.Hq, a.B);
-  kern<<<grid, 192, C::SMEM, stream>>>(tmQ, tmK, tmVt, p, a.window);
+  kern<<<grid, 192, C::SMEM, stream>>>(tmQ, tmK, tmVt, tmQ, tmK, p, a.window, LatentTcParams{});
   count_launch();
   return cudaGetLastError() == cudaSuccess ? nullptr : "flash_fwd_tc launch failed";
 }
 
+// ---- latent attention (models/latent.py): vt[(b, h, d), s] = v[b, s, h, d], zero for d in [vdim, HD) and s >= S
+template <int HD>
+__global__ void transpose_v_latent_kernel(const __nv_bfloat16* __restrict__ v, long long v_bs, long long v_ts, int vdim,
+                                          __nv_bfloat16* __restrict__ vt, int S, int S_pad, int H) {
+  extern __shared__ __nv_bfloat16 tv_tile[];          // [64][HD + 2]
+  const int s0 = blockIdx.x * 64, h = blockIdx.y, b = blockIdx.z;
+  const __nv_bfloat162 zero = __floats2bfloat162_rn(0.f, 0.f);
+  for (int i = threadIdx.x; i < 64 * (HD / 2); i += blockDim.x) {
+    const int r = i / (HD / 2), c2 = i % (HD / 2);
+    __nv_bfloat162 val = zero;
+    if (s0 + r < S && 2 * c2 < vdim)
+      val = *reinterpret_cast<const __nv_bfloat162*>(v + b * v_bs + static_cast<long long>(s0 + r) * v_ts + static_cast<long long>(h) * vdim + 2 * c2);
+    *reinterpret_cast<__nv_bfloat162*>(tv_tile + r * (HD + 2) + 2 * c2) = val;
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < HD * 32; i += blockDim.x) {
+    const int d = i / 32, r2 = i % 32;
+    __nv_bfloat162 val;
+    val.x = tv_tile[(2 * r2) * (HD + 2) + d];
+    val.y = tv_tile[(2 * r2 + 1) * (HD + 2) + d];
+    *reinterpret_cast<__nv_bfloat162*>(vt + ((static_cast<long long>(b) * H + h) * HD + d) * S_pad + s0 + 2 * r2) = val;
+  }
+}
+
+template <int NQ, int HD, int KT>
+const char* launch_latent(const LatentFwdArgs& a, void* vt_ws, int* status, cudaStream_t stream) {
+  using C = Tc3Cfg<NQ, HD, KT>;
+  const int s_pad = (a.S + 63) / 64 * 64;
+  transpose_v_latent_kernel<HD><<<dim3(s_pad / 64, a.heads, a.B), 256, 64 * (HD + 2) * 2, stream>>>(
+      static_cast<const __nv_bfloat16*>(a.v), a.v_bs, a.v_ts, a.vdim, static_cast<__nv_bfloat16*>(vt_ws), a.S, s_pad, a.heads);
+  count_launch();
+  const long long rows = static_cast<long long>(a.B) * a.S;
+  const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q);
+  CUtensorMap tmQ, tmQr, tmK, tmKr, tmVt;
+  if (!make_map_3d(&tmQ, q, rows, a.heads, a.dim, a.dim + a.rot, a.q_ts, FT) ||
+      !make_map_3d(&tmQr, q + a.dim, rows, a.heads, a.rot, a.dim + a.rot, a.q_ts, FT))
+    return "latent_fwd_tc: tensor map for Q failed";
+  if (!make_map_3d(&tmK, a.kn, rows, a.heads, a.dim, a.dim, a.kn_ts, KT) || !make_map_2d(&tmKr, a.kr, rows, a.rot, a.kr_ts, KT))
+    return "latent_fwd_tc: tensor map for K failed";
+  if (!make_map_2d(&tmVt, vt_ws, static_cast<long long>(a.B) * a.heads * HD, s_pad, s_pad, HD))
+    return "latent_fwd_tc: tensor map for V^T failed";
+  FlashTcParams p{};
+  p.out = static_cast<__nv_bfloat16*>(a.out); p.o_bs = a.o_bs; p.o_ts = a.o_ts; p.lse = nullptr;
+  p.B = a.B; p.S = a.S; p.Hq = a.heads; p.Hkv = a.heads; p.scale = a.scale; p.status = status;
+  LatentTcParams lt{};
+  lt.na0 = (a.dim + 63) / 64;
+  lt.vdim = a.vdim;
+  lt.sink = a.sink;
+  for (int ks = 0; ks < (a.dim + 15) / 16; ++ks) lt.kmask |= 1u << ks;
+  for (int ks = 0; ks < (a.rot + 15) / 16; ++ks) lt.kmask |= 1u << (lt.na0 * 4 + ks);
+  auto kern = flash_fwd_tc3_kernel<NQ, HD, KT, true>;
+  if (!FERRL_ONCE_PER_DEVICE(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM) == cudaSuccess))
+    return "latent_fwd_tc: cannot reserve shared memory";
+  kern<<<dim3((a.S + FT - 1) / FT, a.heads, a.B), 192, C::SMEM, stream>>>(tmQ, tmK, tmVt, tmQr, tmKr, p, a.window, lt);
+  count_launch();
+  return cudaGetLastError() == cudaSuccess ? nullptr : "latent_fwd_tc launch failed";
+}
+
+template <int NQ>
+const char* launch_latent_v(const LatentFwdArgs& a, void* vt_ws, int* status, cudaStream_t stream) {
+  constexpr int KT = NQ <= 3 ? 128 : 64;
+  if (a.vdim <= 64) return launch_latent<NQ, 64, KT>(a, vt_ws, status, stream);
+  if (a.vdim <= 128) return launch_latent<NQ, 128, KT>(a, vt_ws, status, stream);
+  return launch_latent<NQ, 256, 64>(a, vt_ws, status, stream);
+}
+
+int latent_atoms(const LatentFwdArgs& a) { return (a.dim + 63) / 64 + (a.rot + 63) / 64; }
+
 }  // namespace
+
+bool latent_fwd_tc_supported(const LatentFwdArgs& a) {
+  auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  const long long S = a.S;
+  return a.dtype == kBF16 && a.S >= 1 && a.dim % 8 == 0 && a.rot % 8 == 0 && a.vdim % 8 == 0 && a.vdim <= 256 && latent_atoms(a) <= 4 &&
+         a.window >= 0 && a.q_bs == S * a.q_ts && a.kn_bs == S * a.kn_ts && a.kr_bs == S * a.kr_ts && a.q_ts % 8 == 0 &&
+         a.kn_ts % 8 == 0 && a.kr_ts % 8 == 0 && a.v_ts % 2 == 0 && a.v_bs % 2 == 0 && a.o_ts % 8 == 0 && a.o_bs % 8 == 0 &&
+         al16(a.q) && al16(a.kn) && al16(a.kr) && al16(a.out) && (reinterpret_cast<uintptr_t>(a.v) & 3) == 0;
+}
+
+size_t latent_fwd_tc_workspace_elems(const LatentFwdArgs& a) {
+  const long long s_pad = (a.S + 63) / 64 * 64, hd = a.vdim <= 64 ? 64 : (a.vdim <= 128 ? 128 : 256);
+  return static_cast<size_t>(a.B) * a.heads * hd * s_pad;
+}
+
+// `vt_ws`: bf16 workspace of latent_fwd_tc_workspace_elems(a) elements, 16-byte aligned
+const char* latent_fwd_tc(const LatentFwdArgs& a, void* vt_ws, int* status, cudaStream_t stream) {
+  if (!latent_fwd_tc_supported(a)) return "latent_fwd_tc: unsupported arguments";
+  if (a.B == 0) return nullptr;
+  switch (latent_atoms(a)) {
+    case 2: return launch_latent_v<2>(a, vt_ws, status, stream);
+    case 3: return launch_latent_v<3>(a, vt_ws, status, stream);
+    default: return launch_latent_v<4>(a, vt_ws, status, stream);
+  }
+}
 
 bool flash_fwd_tc_supported(const FlashArgs& a) {
   auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };

@@ -13,10 +13,9 @@ namespace {
 
 __device__ __forceinline__ float act_fwd(float g, int act) {
   if (act == kActSilu) return g / (1.f + __expf(-g));
-  // gelu tanh approximation
+  // gelu, tanh form: (1 + tanh(u)) / 2 = 1 / (1 + exp(-2u)), which keeps fp32 accuracy under fast math
   const float k0 = 0.7978845608028654f, k1 = 0.044715f;
-  float t = tanhf(k0 * (g + k1 * g * g * g));
-  return 0.5f * g * (1.f + t);
+  return g / (1.f + __expf(-2.f * k0 * (g + k1 * g * g * g)));
 }
 __device__ __forceinline__ float act_grad(float g, int act) {
   if (act == kActSilu) {

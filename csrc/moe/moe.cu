@@ -3,7 +3,7 @@
 // The reference loops over experts on the host and copies the routing table to the host once
 // per layer (crates/ferrl/src/moe.rs:110-158).  Here the whole plan stays on the device:
 //
-//   moe_route_kernel    softmax over E router logits (fp32), top-k, renormalise, count rows/expert
+//   moe_route_kernel    softmax over E router logits or sigmoid of each (fp32), top-k, renormalise, count rows/expert
 //   moe_plan_kernel     stable counting sort of the T*k (token, slot) pairs by expert into
 //                       128-row aligned segments: row_of[pair], token_of[row], tile_expert[m tile]
 //   moe_gather_kernel   xs[row] = scale(row) * x[token_of[row]]   (zero rows for padding)
@@ -31,7 +31,7 @@ constexpr int kSeg = 128;   // segment alignment = GEMM tile height
 
 // One warp per token. logits [T, E] fp32 (row stride ld); E <= 1024.
 __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld, int T, int E, int k, int renorm,
-                                 float* __restrict__ probs, float* __restrict__ scores, int* __restrict__ idx,
+                                 int score, float* __restrict__ probs, float* __restrict__ scores, int* __restrict__ idx,
                                  int* __restrict__ counts) {
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   const int lane = threadIdx.x & 31;
@@ -48,11 +48,12 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, long long ld,
   mx = warp_max(mx);
   float sum = 0.f;
   for (int i = 0; i < per; ++i) {
-    v[i] = (i * 32 + lane < E) ? __expf(v[i] - mx) : 0.f;
+    if (score == 1) v[i] = (i * 32 + lane < E) ? 1.f / (1.f + __expf(-v[i])) : 0.f;
+    else v[i] = (i * 32 + lane < E) ? __expf(v[i] - mx) : 0.f;
     sum += v[i];
   }
   sum = warp_sum(sum);
-  const float inv = 1.f / sum;
+  const float inv = score == 1 ? 1.f : 1.f / sum;
   for (int i = 0; i < per; ++i) {
     v[i] *= inv;
     const int e = i * 32 + lane;
@@ -231,15 +232,124 @@ __global__ void moe_pair_dot_kernel(const __nv_bfloat16* __restrict__ dy, const 
   if (lane == 0) dw[pair] = acc;
 }
 
+// ---- any type and size
+template <typename T>
+__global__ void moe_gather_any_kernel(const T* __restrict__ x, long long ldx, const int* __restrict__ token_of,
+                                      const float* __restrict__ row_scale, int rows, int H, T* __restrict__ xs) {
+  const long long n = static_cast<long long>(rows) * H;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < n;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const int r = static_cast<int>(i / H), c = static_cast<int>(i - static_cast<long long>(r) * H);
+    const int t = token_of[r];
+    float v = 0.f;
+    if (t >= 0) v = to_f(x[t * ldx + c]) * (row_scale ? row_scale[r] : 1.f);
+    xs[i] = from_f<T>(v);
+  }
+}
+template <typename T>
+__global__ void moe_combine_any_kernel(const T* __restrict__ ys, const int* __restrict__ row_of, const float* __restrict__ w,
+                                       int tokens, int k, int H, T* __restrict__ out) {
+  const long long n = static_cast<long long>(tokens) * H;
+  for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < n;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const int t = static_cast<int>(i / H), c = static_cast<int>(i - static_cast<long long>(t) * H);
+    float acc = 0.f;
+    for (int j = 0; j < k; ++j) {
+      const long long p = static_cast<long long>(t) * k + j;
+      acc += (w ? w[p] : 1.f) * to_f(ys[static_cast<long long>(row_of[p]) * H + c]);
+    }
+    out[i] = from_f<T>(acc);
+  }
+}
+// 32 x 32 output tile per CTA of 256 threads, four rows a thread, fp32 multiply-add
+template <typename T>
+__global__ void moe_grouped_any_kernel(const T* __restrict__ xs, const T* __restrict__ W, const int* __restrict__ tile_expert,
+                                       int N, int K, T* __restrict__ out) {
+  __shared__ float sx[32][33], sw[32][33];
+  const int n0 = blockIdx.x * 32, r0 = blockIdx.y * 32;
+  const int e = tile_expert[r0 / kSeg];
+  if (e < 0) return;
+  const T* we = W + static_cast<long long>(e) * N * K;
+  const int tx = threadIdx.x & 31, ty = threadIdx.x >> 5;
+  float acc[4] = {0.f, 0.f, 0.f, 0.f};
+  for (int k0 = 0; k0 < K; k0 += 32) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int r = ty + i * 8, k = k0 + tx;
+      sx[r][tx] = k < K ? to_f(xs[static_cast<long long>(r0 + r) * K + k]) : 0.f;
+      sw[r][tx] = (k < K && n0 + r < N) ? to_f(we[static_cast<long long>(n0 + r) * K + k]) : 0.f;
+    }
+    __syncthreads();
+    for (int k = 0; k < 32; ++k) {
+      const float b = sw[tx][k];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[i] += sx[ty + i * 8][k] * b;
+    }
+    __syncthreads();
+  }
+  if (n0 + tx < N) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) out[static_cast<long long>(r0 + ty + i * 8) * N + n0 + tx] = from_f<T>(acc[i]);
+  }
+}
+
+unsigned any_grid(long long n) { return static_cast<unsigned>(std::min<long long>((n + 255) / 256, 148 * 16)); }
+
 }  // namespace
 
-const char* moe_route(const float* logits, long long ld, int T, int E, int k, bool renorm, float* probs, float* scores,
-                      int* idx, int* counts, cudaStream_t stream) {
+const char* moe_gather_any(int dtype, const void* x, long long ldx, const int* token_of, const float* pair_w, const int* row_of,
+                           int n_pairs, float* row_scale, int rows, int H, void* xs, cudaStream_t stream) {
+  if (pair_w) {
+    moe_row_scale_kernel<<<(n_pairs + 255) / 256, 256, 0, stream>>>(pair_w, row_of, n_pairs, row_scale);
+    count_launch();
+  }
+  const unsigned grid = any_grid(static_cast<long long>(rows) * H);
+  const float* rs = pair_w ? row_scale : nullptr;
+  if (dtype == kF32)
+    moe_gather_any_kernel<float><<<grid, 256, 0, stream>>>(static_cast<const float*>(x), ldx, token_of, rs, rows, H, static_cast<float*>(xs));
+  else
+    moe_gather_any_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(static_cast<const __nv_bfloat16*>(x), ldx, token_of, rs, rows, H,
+                                                                   static_cast<__nv_bfloat16*>(xs));
+  count_launch();
+  return cudaGetLastError() == cudaSuccess ? nullptr : "moe_gather_any launch failed";
+}
+
+const char* moe_grouped_any(int dtype, const void* xs, const void* W, const int* tile_expert, int rows, int N, int K, void* out,
+                            cudaStream_t stream) {
+  if (rows % kSeg || rows / 32 > 65535) return "moe_grouped_any: rows in 128-row segments, at most 2 M of them";
+  if (rows == 0) return nullptr;
+  const dim3 grid((N + 31) / 32, rows / 32);
+  if (dtype == kF32)
+    moe_grouped_any_kernel<float><<<grid, 256, 0, stream>>>(static_cast<const float*>(xs), static_cast<const float*>(W), tile_expert, N, K,
+                                                            static_cast<float*>(out));
+  else
+    moe_grouped_any_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(static_cast<const __nv_bfloat16*>(xs),
+                                                                    static_cast<const __nv_bfloat16*>(W), tile_expert, N, K,
+                                                                    static_cast<__nv_bfloat16*>(out));
+  count_launch();
+  return cudaGetLastError() == cudaSuccess ? nullptr : "moe_grouped_any launch failed";
+}
+
+const char* moe_combine_any(int dtype, const void* ys, const int* row_of, const float* w, int T, int k, int H, void* out,
+                            cudaStream_t stream) {
+  if (T == 0) return nullptr;
+  const unsigned grid = any_grid(static_cast<long long>(T) * H);
+  if (dtype == kF32)
+    moe_combine_any_kernel<float><<<grid, 256, 0, stream>>>(static_cast<const float*>(ys), row_of, w, T, k, H, static_cast<float*>(out));
+  else
+    moe_combine_any_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(static_cast<const __nv_bfloat16*>(ys), row_of, w, T, k, H,
+                                                                    static_cast<__nv_bfloat16*>(out));
+  count_launch();
+  return cudaGetLastError() == cudaSuccess ? nullptr : "moe_combine_any launch failed";
+}
+
+const char* moe_route(const float* logits, long long ld, int T, int E, int k, bool renorm, int score, float* probs,
+                      float* scores, int* idx, int* counts, cudaStream_t stream) {
   if (E > 1024 || k > kMaxTopK || k > E || k > 32) return "moe_route: E <= 1024 and k <= 16 supported";
   if (T == 0) return nullptr;
   cudaMemsetAsync(counts, 0, sizeof(int) * E, stream);
   const int threads = 256, warps = threads / 32;
-  moe_route_kernel<<<(T + warps - 1) / warps, threads, 0, stream>>>(logits, ld, T, E, k, renorm ? 1 : 0, probs, scores,
+  moe_route_kernel<<<(T + warps - 1) / warps, threads, 0, stream>>>(logits, ld, T, E, k, renorm ? 1 : 0, score, probs, scores,
                                                                    idx, counts);
   count_launch();
   return cudaGetLastError() == cudaSuccess ? nullptr : "moe_route launch failed";

@@ -102,10 +102,14 @@ def routed_experts(x: torch.Tensor, logits: torch.Tensor, gate_up, down, top_k: 
                    renorm: bool = True, weight_input: bool = False, act: str = "silu") -> torch.Tensor:
     """Experts behind router logits computed elsewhere (float32 ``[T, E]``): the device-resident plan on GPUs, the
     eager one on the CPU.  ``x`` ``[T, H]``."""
-    if ops_native(x) and not (gate_up.requires_grad or down.requires_grad):
+    if ops_native(x) and gate_up.shape[0] <= 1024 and top_k <= 16:
         from ..ops import cuda as C
         scores, idx, counts, _ = C.moe_route(logits, top_k, renorm, score)
-        return C.moe_experts(x, scores, idx, counts, gate_up, down, act, weight_input=weight_input)
+        y = C.moe_experts(x, scores, idx, counts, gate_up, down, act, weight_input=weight_input)
+        if y is None and not (torch.is_grad_enabled() and any(t.requires_grad for t in (x, logits, gate_up, down))):
+            y = C.moe_experts_any(x, scores, idx, counts, gate_up, down, act, weight_input)
+        if y is not None:
+            return y
     _, scores, idx = topk_scores(logits, top_k, renorm, score)
     return moe_experts(x, idx, scores, gate_up, down, act, weight_input)
 

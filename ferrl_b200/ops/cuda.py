@@ -107,7 +107,7 @@ class _LoraLinear(torch.autograd.Function):
     def forward(ctx, x, w, wt, a_stack, b_stack, residual=None):
         K = x.shape[-1]
         x2 = x.reshape(-1, K)
-        if not x2.is_contiguous():
+        if x2.stride(1) != 1 or x2.stride(0) % 8 or x2.data_ptr() % 16:      # rows of a wider tensor are read in place
             x2 = x2.contiguous()
         t = a16 = b16 = None
         if a_stack is not None:
@@ -531,6 +531,111 @@ def kv_append(k_cache, v_cache, k, v, kv_len):
         (B, v.shape[-2] * v.shape[-1]), (v.stride(0), 1), v.storage_offset()), k_cache, v_cache, kv_len)
 
 
+# ------------------------------------------------------- latent attention, post-norm layers
+class _EagerGrad(torch.autograd.Function):
+    """Native forward with the eager restatement's gradient: ``backward`` replays ``eager_fn`` on the saved tensors."""
+
+    @staticmethod
+    def forward(ctx, native_fn, eager_fn, *tensors):
+        ctx.eager_fn = eager_fn
+        ctx.present = [t is not None for t in tensors]
+        ctx.save_for_backward(*[t for t in tensors if t is not None])
+        return native_fn(*tensors)
+
+    @staticmethod
+    def backward(ctx, *gout):
+        saved = iter(ctx.saved_tensors)
+        ins = [next(saved).detach().requires_grad_(ctx.needs_input_grad[2 + i]) if p else None
+               for i, p in enumerate(ctx.present)]
+        with torch.enable_grad():
+            out = ctx.eager_fn(*ins)
+        outs = out if isinstance(out, tuple) else (out,)
+        pairs = [(o, g) for o, g in zip(outs, gout) if g is not None and o.requires_grad]
+        wanted = [t for t in ins if t is not None and t.requires_grad]
+        grads = iter(torch.autograd.grad([o for o, _ in pairs], wanted, [g for _, g in pairs], allow_unused=True))
+        return (None, None) + tuple(next(grads) if t is not None and t.requires_grad else None for t in ins)
+
+
+def _wants_grad(*ts):
+    return torch.is_grad_enabled() and any(t is not None and t.requires_grad for t in ts)
+
+
+def _rows2(t, W):
+    t = t.reshape(-1, W)
+    return t if t.stride(1) == 1 else t.contiguous()
+
+
+def post_norm(x, y, weight, bias, eps, alpha, gate, gate_bias, history, coef, cast, out):
+    """See ``csrc/kernels/post_norm.cu``; with gradients the forward is the same kernel and the backward eager."""
+    def native_fn(x_, y_, w_, b_, g_, gb_, h_, c_):
+        W = x_.shape[-1]
+        nxt, low, r = lib().post_norm(x_.contiguous(), None if y_ is None else _rows2(y_, W), None if g_ is None else _rows2(g_, W),
+                                      gb_, w_, b_, float(eps), float(alpha), h_, c_, cast == torch.bfloat16, out)
+        return nxt, low, r
+    args = (x, y, weight, bias, gate, gate_bias, history, coef)
+    if _wants_grad(*args):
+        def eager_fn(x_, y_, w_, b_, g_, gb_, h_, c_):
+            return eager.post_norm(x_, y_, w_, b_, eps, alpha, g_, gb_, h_, c_)[0]
+        nxt = _EagerGrad.apply(lambda *a: native_fn(*a)[0], eager_fn, *args)
+        return nxt, nxt if cast is None else nxt.to(cast), nxt
+    nxt, low, r = native_fn(*args)
+    return nxt, nxt if cast is None else low, r
+
+
+def _latent_views(q, dkv):
+    """``[n_tok, H, E]`` and ``[n_tok, rank + rot]`` views of (possibly strided) projections."""
+    E = q.shape[-1]
+    if q.stride(-1) != 1 or q.stride(-2) != E:
+        q = q.contiguous()
+    if dkv.stride(-1) != 1:
+        dkv = dkv.contiguous()
+    return q.reshape(-1, q.shape[-2], E), dkv.reshape(-1, dkv.shape[-1])
+
+
+def latent_prep(q, dkv, norm_w, eps, cos, sin, positions, dim, rank):
+    if _wants_grad(q, dkv, norm_w):
+        return eager.latent_prep(q, dkv, norm_w, eps, cos, sin, positions, dim, rank)
+    q3, d2 = _latent_views(q, dkv)
+    width = eager.latent_row_width(rank, q.shape[-1] - dim)
+    rows = lib().latent_prep(q3, d2, norm_w, float(eps), cos, sin, positions.contiguous(), dim, rank, width)
+    same = q3.data_ptr() == q.data_ptr()
+    return (q if same else q3.view(q.shape)), rows.view(*q.shape[:-2], width)
+
+
+def latent_append(q, dkv, norm_w, eps, cos, sin, kv_len, cache, dim, rank):
+    q3, d2 = _latent_views(q, dkv)
+    lib().latent_append(q3, d2, norm_w, float(eps), cos, sin, kv_len, cache, dim, rank)
+    return q3
+
+
+def latent_attention(q, kv, lat, *, dim, vdim, rank, scale, window=0, sink=None, variant=0):
+    """Whole sequences: tcgen05 where the sizes fit (``csrc/kernels/flash_tc.cu``), the any-size kernel otherwise
+    (``variant=1`` forces it)."""
+    def native_fn(q_, kv_, lat_, s_):
+        q_ = q_ if (q_.stride(3) == 1 and q_.stride(2) == q_.shape[3]) else q_.contiguous()
+        return lib().latent_fwd(q_, kv_ if kv_.stride(2) == 1 else kv_.contiguous(), lat_ if lat_.stride(2) == 1 else lat_.contiguous(),
+                                dim, vdim, rank, float(scale), int(window or 0), s_, int(variant))
+    if _wants_grad(q, kv, lat, sink):
+        return _EagerGrad.apply(native_fn, lambda q_, kv_, lat_, s_: eager.latent_attention(
+            q_, kv_, lat_, dim=dim, vdim=vdim, rank=rank, scale=scale, window=window, sink=s_), q, kv, lat, sink)
+    return native_fn(q, kv, lat, sink)
+
+
+def latent_decode(q, uk_t, uv, cache, count, *, rank, scale, sink=None, splits=0):
+    """``splits`` forces the number of key ranges per row (0: planned from the batch)."""
+    return lib().latent_decode(q, uk_t, uv if uv.is_contiguous() else uv.contiguous(), cache, count, float(scale), sink, int(splits))
+
+
+def linear_f32(x, w):
+    """float32 result of a projection: tcgen05 GEMM with an fp32 epilogue for bf16 operands."""
+    if _wants_grad(x, w) or not (_bf16(x) and _bf16(w)) or x.shape[-1] % 8:
+        return eager.linear_f32(x, w)
+    x2 = x.reshape(-1, x.shape[-1])
+    if x2.shape[0] == 0:
+        return torch.empty(*x.shape[:-1], w.shape[0], dtype=torch.float32, device=x.device)
+    return gemm(x2 if x2.is_contiguous() else x2.contiguous(), w, out_f32=True, static_b=True).view(*x.shape[:-1], w.shape[0])
+
+
 # ------------------------------------------------------------------ mlp
 _ACT = {"silu": 0, "gelu_pytorch_tanh": 1, "gelu_tanh": 1}
 
@@ -658,14 +763,15 @@ def gdn_decode_step_raw(q, k, v, a, b, A_log, dt_bias, S, l2norm=True, eps=1e-6)
 
 # ------------------------------------------------------------------ MoE
 class _MoeRoute(torch.autograd.Function):
-    """fp32 softmax over the router logits, top-k and renormalisation in one kernel; the
-    backward is the closed form of softmax -> gather -> normalise on the small [T, E] table."""
+    """fp32 scores (softmax over the router logits, or the sigmoid of each), top-k and renormalisation in one
+    kernel; the backward is the closed form of score -> gather -> normalise on the small [T, E] table."""
 
     @staticmethod
-    def forward(ctx, logits, k, renorm):
-        probs, scores, idx, counts = lib().moe_route(logits.contiguous(), k, renorm)
+    def forward(ctx, logits, k, renorm, score):
+        probs, scores, idx, counts = lib().moe_route(logits if logits.stride(1) == 1 else logits.contiguous(), k, renorm,
+                                                     1 if score == "sigmoid" else 0)
         ctx.save_for_backward(probs, scores, idx)
-        ctx.renorm = renorm
+        ctx.renorm, ctx.score = renorm, score
         ctx.mark_non_differentiable(idx, counts)
         return scores, idx, counts, probs.detach()
 
@@ -677,24 +783,31 @@ class _MoeRoute(torch.autograd.Function):
             top = probs.gather(1, li).sum(-1, keepdim=True)
             ds = (ds - (ds * scores).sum(-1, keepdim=True)) / top
         dp = torch.zeros_like(probs).scatter_(1, li, ds)
-        return probs * (dp - (dp * probs).sum(-1, keepdim=True)), None, None
+        if ctx.score == "sigmoid":
+            return dp * probs * (1.0 - probs), None, None, None
+        return probs * (dp - (dp * probs).sum(-1, keepdim=True)), None, None, None
 
 
-def moe_route(logits_f32, k, renorm=True):
-    """``(scores [T,k] f32, idx [T,k] i32, counts [E] i32, probs [T,E] f32)``."""
-    return _MoeRoute.apply(logits_f32, int(k), bool(renorm))
+def moe_route(logits_f32, k, renorm=True, score="softmax"):
+    """``(scores [T,k] f32, idx [T,k] i32, counts [E] i32, probs [T,E] f32)``; ``score`` is ``softmax`` over the
+    experts or ``sigmoid`` of each."""
+    if score not in ("softmax", "sigmoid"):
+        raise ValueError(f"unknown routing score {score!r}")
+    return _MoeRoute.apply(logits_f32, int(k), bool(renorm), score)
 
 
 class _MoeExperts(torch.autograd.Function):
     """Routed frozen experts: plan -> gather -> grouped GEMM -> SwiGLU -> grouped GEMM -> combine,
-    with no host synchronisation; gradients flow to the tokens and to the routing scores."""
+    with no host synchronisation; gradients flow to the tokens and to the routing scores.  The routing weights
+    multiply the experts' outputs, or (``weight_input``) their inputs while the rows are gathered."""
 
     @staticmethod
-    def forward(ctx, x, scores, idx, counts, gate_up, down, gate_up_t, down_t, act):
+    def forward(ctx, x, scores, idx, counts, gate_up, down, gate_up_t, down_t, act, weight_input=False):
         L = lib()
         T, k = idx.shape
+        sc = scores.float().contiguous()
         row_of, token_of, tile_expert, _ = L.moe_plan(idx.contiguous(), counts)
-        xs = L.moe_gather(x.contiguous(), token_of, None, row_of)
+        xs = L.moe_gather(x.contiguous(), token_of, sc if weight_input else None, row_of)
         # rows of unused tiles are never written and never read back (the combine reads routed rows only); the
         # zero fill of the outputs is kept for training, where the padded rows are saved for the backward pass
         train = any(ctx.needs_input_grad)
@@ -705,10 +818,10 @@ class _MoeExperts(torch.autograd.Function):
         o2 = None if train else torch.empty(h.shape[0], down.shape[1], dtype=h.dtype, device=h.device)
         ys = L.moe_grouped_gemm(h, down, tile_expert, o2)
         del h
-        sc = scores.float().contiguous()
-        out = L.moe_combine(ys, row_of, sc, T, k)
-        ctx.save_for_backward(gu, ys, sc, row_of, token_of, tile_expert, gate_up, down, gate_up_t, down_t)
-        ctx.act, ctx.k = act, k
+        out = L.moe_combine(ys, row_of, None if weight_input else sc, T, k)
+        # kept rows: the outputs for the gradient of output weights, the tokens for that of input weights
+        ctx.save_for_backward(gu, x if weight_input else ys, sc, row_of, token_of, tile_expert, gate_up, down, gate_up_t, down_t)
+        ctx.act, ctx.k, ctx.weight_input = act, k, weight_input
         ctx.score_dtype = scores.dtype
         return out
 
@@ -718,8 +831,10 @@ class _MoeExperts(torch.autograd.Function):
         gu, ys, sc, row_of, token_of, tile_expert, gate_up, down, gate_up_t, down_t = ctx.saved_tensors
         dout = dout.contiguous()
         T = dout.shape[0]
-        dsc = L.moe_pair_dot(dout, ys, row_of, ctx.k).to(ctx.score_dtype)
-        dys = L.moe_gather(dout, token_of, sc.view(-1), row_of)
+        dsc = None
+        if not ctx.weight_input:
+            dsc = L.moe_pair_dot(dout, ys, row_of, ctx.k).to(ctx.score_dtype)
+        dys = L.moe_gather(dout, token_of, None if ctx.weight_input else sc.view(-1), row_of)
         if down_t is None:
             down_t = down.transpose(1, 2).contiguous()
         dh = L.moe_grouped_gemm(dys, down_t, tile_expert)
@@ -729,11 +844,19 @@ class _MoeExperts(torch.autograd.Function):
         if gate_up_t is None:
             gate_up_t = gate_up.transpose(1, 2).contiguous()
         dxs = L.moe_grouped_gemm(dgu, gate_up_t, tile_expert)
-        dx = L.moe_combine(dxs, row_of, None, T, ctx.k)
-        return dx, dsc, None, None, None, None, None, None, None
+        if ctx.weight_input:
+            dsc = L.moe_pair_dot(ys.contiguous(), dxs, row_of, ctx.k).to(ctx.score_dtype)     # <token, d(weighted token)>
+        dx = L.moe_combine(dxs, row_of, sc if ctx.weight_input else None, T, ctx.k)
+        return dx, dsc, None, None, None, None, None, None, None, None
 
 
-def moe_experts(x, scores, idx, counts, gate_up, down, act="silu", gate_up_t=None, down_t=None):
+def moe_experts_any(x, scores, idx, counts, gate_up, down, act="silu", weight_input=False):
+    """Grad-free routed experts for fp32 and for sizes outside ``moe_experts``'s domain, on the same device plan."""
+    return lib().moe_experts_any(x if x.stride(1) == 1 else x.contiguous(), scores.float().contiguous(), idx.contiguous(), counts, gate_up, down,
+                                 _ACT[act], bool(weight_input))
+
+
+def moe_experts(x, scores, idx, counts, gate_up, down, act="silu", gate_up_t=None, down_t=None, weight_input=False):
     """``x`` ``[T,H]`` bf16; ``gate_up`` ``[E,2I,H]``, ``down`` ``[E,H,I]`` frozen bf16; optional
     resident transposes for the backward GEMMs.  ``None`` when the shapes are outside the kernels'
     domain (caller falls back to the eager plan)."""
@@ -742,7 +865,7 @@ def moe_experts(x, scores, idx, counts, gate_up, down, act="silu", gate_up_t=Non
     H, I = x.shape[-1], down.shape[-1]
     if H % 8 or I % 8 or not (gate_up.is_contiguous() and down.is_contiguous()):
         return None
-    return _MoeExperts.apply(x, scores, idx, counts, gate_up, down, gate_up_t, down_t, _ACT[act])
+    return _MoeExperts.apply(x, scores, idx, counts, gate_up, down, gate_up_t, down_t, _ACT[act], bool(weight_input))
 
 
 def embedding(ids, table, scale=1.0):

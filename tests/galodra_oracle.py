@@ -47,46 +47,50 @@ def layer_norm(x, w, b, eps):
 
 def rotate(x, positions, dims, base):
     """Rotate-half on the first ``dims`` entries of the last axis of ``x`` ``[T, ..., D]``."""
-    out = x.clone()
+    cols = [x[..., i] for i in range(x.shape[-1])]
     for i in range(dims // 2):
         f = base ** (-2.0 * i / dims)
-        for t, p in enumerate(positions):
-            c, s = math.cos(p * f), math.sin(p * f)
-            u, v = x[t, ..., i].clone(), x[t, ..., i + dims // 2].clone()
-            out[t, ..., i] = u * c - v * s
-            out[t, ..., i + dims // 2] = v * c + u * s
-    return out
+        shape = [-1] + [1] * (x.dim() - 2)
+        c = torch.tensor([math.cos(p * f) for p in positions], dtype=x.dtype).view(shape)
+        s = torch.tensor([math.sin(p * f) for p in positions], dtype=x.dtype).view(shape)
+        u, v = x[..., i], x[..., i + dims // 2]
+        cols[i], cols[i + dims // 2] = u * c - v * s, v * c + u * s
+    return torch.stack(cols, -1)
 
 
 def sink_softmax(scores, sink):
-    """Weights over a list of scores whose denominator also holds ``exp(sink)``."""
-    m = max(float(scores.max()), float(sink))
-    e = torch.exp(scores - m)
-    return e / (e.sum() + math.exp(float(sink) - m))
+    """Weights over the last axis of ``scores`` ``[H, n]`` whose denominators also hold ``exp(sink[h])``."""
+    m = torch.maximum(scores.max(-1).values, sink).detach()
+    e = torch.exp(scores - m[:, None])
+    return e / (e.sum(-1) + torch.exp(sink - m))[:, None]
 
 
 def visible(i, window):
-    return range(max(0, i - window + 1), i + 1)
+    return list(range(max(0, i - window + 1), i + 1))
+
+
+def attend(qn, qr, kn, kr, v, scale, window, sink):
+    """``qn`` ``[T,H,D]``, ``qr`` ``[T,H,R]``, ``kn`` ``[T,H,D]``, ``kr`` ``[T,R]``, ``v`` ``[T,H,V]`` -> ``[T,H,V]``."""
+    rows = []
+    for i in range(qn.shape[0]):
+        js = visible(i, window)
+        s = (torch.einsum("hd,jhd->hj", qn[i], kn[js]) + torch.einsum("hr,jr->hj", qr[i], kr[js])) * scale
+        rows.append(torch.einsum("hj,jhv->hv", sink_softmax(s, sink), v[js]))
+    return torch.stack(rows)
 
 
 def latent_attention(h, w, p, mx, eps):
     """``h`` ``[T, width]``; ``p`` is the tensor prefix, ``mx`` the mixer's configuration."""
     H, D, R, V, K = mx["heads"], mx["dim"], mx["rot_dim"], mx["vdim"], mx["kv_rank"]
-    T = h.shape[0]
+    T, rot = h.shape[0], mx["rot"]
     q = (h @ w[p + "q"].T).reshape(T, H, D + R)
-    qn, qr = q[..., :D], rotate(q[..., D:], range(T), mx["rot"]["dims"], mx["rot"]["base"])
     kv = h @ w[p + "dkv"].T
     c = rms_norm(kv[:, :K], w[p + "dkv.norm"], eps)
-    kr = rotate(kv[:, K:], range(T), mx["rot"]["dims"], mx["rot"]["base"])
     kn = (c @ w[p + "uk"].T).reshape(T, H, D)
     v = (c @ w[p + "uv"].T).reshape(T, H, V)
-    out = torch.zeros(T, H, V, dtype=h.dtype)
-    for i in range(T):
-        js = list(visible(i, mx["mask"]["size"]))
-        for a in range(H):
-            s = (kn[js, a] @ qn[i, a] + kr[js] @ qr[i, a]) * mx["scale"]
-            out[i, a] = sink_softmax(s, w[p + "sink"][a]) @ v[js, a]
-    return out.reshape(T, H * V) @ w[p + "o"].T
+    o = attend(q[..., :D], rotate(q[..., D:], range(T), rot["dims"], rot["base"]), kn,
+               rotate(kv[:, K:], range(T), rot["dims"], rot["base"]), v, mx["scale"], mx["mask"]["size"], w[p + "sink"])
+    return o.reshape(T, H * V) @ w[p + "o"].T
 
 
 def dense_ff(h, w, p):
@@ -98,7 +102,7 @@ def route(h, w, p, top):
     s = 1 / (1 + torch.exp(-(h @ w[p + "router"].T)))
     picks = []
     for t in range(h.shape[0]):
-        order = sorted(range(s.shape[1]), key=lambda e: (-float(s[t, e]), e))[:top]
+        order = sorted(range(s.shape[1]), key=lambda e: (-s[t, e].item(), e))[:top]
         picks.append([(e, s[t, e]) for e in order])
     return picks
 
@@ -108,11 +112,10 @@ def expert(h, w, p):
 
 
 def moe_ff(h, w, p, top):
-    out = torch.zeros_like(h)
+    rows = []
     for t, pick in enumerate(route(h, w, p, top)):
-        for e, s in pick:
-            out[t] += expert(s * h[t], w, f"{p}e{e}.")
-    return out
+        rows.append(sum(expert(s * h[t], w, f"{p}e{e}.") for e, s in pick))
+    return torch.stack(rows)
 
 
 def residual_gate(h, w, name):
@@ -142,7 +145,7 @@ def layer(x, w, i, lc, cfg):
 
 def forward(tokens, weights, cfg, dt=torch.float64, layers_out=None):
     """Logits ``[T, vocab]`` of one sequence."""
-    w = {k: v.to(dt) if v.is_floating_point() else v for k, v in weights.items()}
+    w = {k: v.to(dt) for k, v in weights.items()}
     x = w["embed"][list(tokens)]
     history = [x]
     for i, lc in enumerate(cfg["layers"]):

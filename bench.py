@@ -238,7 +238,14 @@ def main():
     ap.add_argument("--seed", type=int, default=1234)
     ap.add_argument("--no-graph", action="store_true", help="run decode steps eagerly (for per-kernel profiling)")
     ap.add_argument("--nccl-baseline", action="store_true", help="use per-tensor NCCL all-reduce instead of the fused DP step")
+    ap.add_argument("--serving", nargs="?", const="all", default=None,
+                    help="instead of the training step: prefill and decode throughput of the Galodra family beside the closest "
+                         "existing one (dense-4k, dense-1k, moe-2k, comma-separated, or all); see bench_serving.py")
     args = ap.parse_args()
+    if args.serving is not None:
+        import bench_serving
+        names = list(bench_serving.SIZES) if args.serving == "all" else args.serving.split(",")
+        return bench_serving.main(names, max(args.steps, 10), max(args.warmup, 3), ClockSampler)
     for k in ("prompts", "group", "max_new", "prompt_lo", "prompt_hi", "microbatch", "remat"):
         if getattr(args, k) is None:
             setattr(args, k, CONFIGS[args.config][k])

@@ -196,6 +196,76 @@ def profile_case(name, C):
     return 0
 
 
+def latent_kernels(C, T, report, dev):
+    """Kernels of the latent-attention / post-norm layers, each beside the like kernel of the existing families."""
+    from ferrl_b200 import ops
+    bf = torch.bfloat16
+    rnd = lambda *s: torch.randn(*s, device=dev, dtype=bf)  # noqa: E731
+    pairs = lambda S, w: sum(min(i + 1, w) for i in range(S))  # noqa: E731
+    with torch.no_grad():
+        for B, S, w in ((8, 2048, 1024), (8, 2048, 2048)):
+            for H, D, R, V, K in ((32, 128, 64, 128, 512), (16, 64, 32, 64, 256)):
+                q, kv, lat = rnd(B, S, H, D + R), rnd(B, S, H * (D + V)), rnd(B, S, K + R)
+                sink = torch.randn(H, device=dev)
+                s = T(lambda: C.latent_attention(q, kv, lat, dim=D, vdim=V, rank=K, scale=0.07, window=w, sink=sink))
+                report(f"latent prefill B{B} S{S} w{w} H{H} {D}+{R}/{V}", s, 0, 2 * B * H * pairs(S, w) * (D + R + V))
+            for H, Hk, D in ((32, 16, 128), (16, 8, 64), (16, 2, 256)):
+                q, k, v = rnd(B, S, H, D), rnd(B, S, Hk, D), rnd(B, S, Hk, D)
+                s = T(lambda: C.attention(q, k, v, scale=0.07, causal=True, window=w if w < S else 0))
+                report(f"  flash prefill B{B} S{S} w{w} {H}q/{Hk}kv d{D}", s, 0, 4 * B * H * pairs(S, w) * D)
+        for B, slots in ((128, 1024), (16, 1024), (128, 4096)):
+            for H, D, R, V, K in ((32, 128, 64, 128, 512), (16, 128, 64, 128, 512), (64, 128, 64, 128, 512), (16, 64, 32, 64, 256)):
+                q, uk, uv, cache = rnd(B, H, D + R), rnd(H, K, D), rnd(H, V, K), rnd(B, slots, K + R)
+                cnt, one = (torch.full((B,), n, device=dev, dtype=torch.int32) for n in (slots, 1))
+                sink = torch.randn(H, device=dev)
+                s = T(lambda: C.latent_decode(q, uk, uv, cache, cnt, rank=K, scale=0.07, sink=sink))
+                s1 = T(lambda: C.latent_decode(q, uk, uv, cache, one, rank=K, scale=0.07, sink=sink, splits=1))
+                by = B * slots * (K + R) * 2
+                report(f"latent decode B{B} slots{slots} H{H} {K}+{R}", s, by + (uk.numel() + uv.numel()) * 2, 2 * B * slots * H * (2 * K + R),
+                       f"with absorption; {s1 * 1e6:.1f} us of it without keys")
+                if B == 128 and slots == 1024:
+                    for n in (1, 2, 4):
+                        s = T(lambda: C.latent_decode(q, uk, uv, cache, cnt, rank=K, scale=0.07, sink=sink, splits=n))
+                        report(f"   splits {n}", s, by, 0)
+            for H, Hk, D in ((32, 16, 128), (32, 8, 128), (16, 8, 64), (16, 2, 256)):
+                if B * slots * Hk * D > 1 << 31:
+                    continue
+                q, k, v = rnd(B, H, D), rnd(B, slots, Hk, D), rnd(B, slots, Hk, D)
+                cnt = torch.full((B,), slots, device=dev, dtype=torch.int32)
+                s = T(lambda: C.decode_attention(q, k, v, cnt, scale=0.07))
+                report(f"  decode attention B{B} len{slots} {H}q/{Hk}kv d{D}", s, 2 * B * slots * Hk * D * 2, 0)
+        cos, sin = (t.to(dev) for t in ops.rope_tables(ops.default_inv_freq(64, 1e4), 4096))
+        H, D, R, K, W = 32, 128, 64, 512, 4096
+        nq = H * (D + R)
+        fused, nw, pos = rnd(8, 2048, nq + K + R + W), torch.ones(K, device=dev), torch.arange(2048, device=dev)
+        views = lambda f: (f[..., :nq].unflatten(-1, (H, D + R)), f[..., nq:nq + K + R])  # noqa: E731
+        n = 8 * 2048
+        s = T(lambda: C.latent_prep(*views(fused), nw, 1e-6, cos, sin, pos, D, K))
+        report("latent prep 16384 tokens H32 512+64", s, n * 2 * (2 * (K + R) + 2 * H * R), 0)
+        c128, s128 = (t.to(dev) for t in ops.rope_tables(ops.default_inv_freq(128, 1e4), 4096))
+        q, k, w128 = rnd(8, 2048, 32, 128), rnd(8, 2048, 16, 128), torch.ones(128, device=dev, dtype=bf)
+        s = T(lambda: C.qk_norm_rope(q, k, w128, w128, 1e-6, c128, s128, pos))
+        report("  qk norm + rope 16384 tokens 32q/16kv", s, n * 2 * 2 * 48 * 128, 0)
+        for rows in (16384, 128):
+            x, y, g = torch.randn(rows, W, device=dev), rnd(rows, W), rnd(rows, W)
+            v1, xb = torch.ones(W, device=dev), rnd(rows, W)
+            for h in (0, 1, 8, 32):
+                if rows * h * W * 4 > 3 << 30:
+                    continue
+                hist, coef = (torch.randn(h, rows, W, device=dev), torch.ones(h + 1, device=dev)) if h else (None, None)
+                out = torch.empty(rows, W, device=dev) if h else None
+                s = T(lambda: C.post_norm(x, y, v1, v1, 1e-6, 2.0, g, v1, hist, coef, bf, out))
+                report(f"post norm {rows} rows W4096 history {h}", s, rows * W * (4 + 2 + 2 + 4 + 2 + (4 * h + 4 if h else 0)), 0)
+            wb = torch.ones(W, device=dev, dtype=bf)
+            s = T(lambda: C.add_rmsnorm(xb, y, wb, 1e-6))
+            report(f"  add + rmsnorm {rows} rows W4096", s, rows * W * 2 * 4, 0)
+        lg = torch.randn(16384, 64, device=dev)
+        s = T(lambda: C.moe_route(lg, 8, False, "sigmoid"))
+        report("moe route sigmoid 16384 x 64 top 8", s, 16384 * (64 * 8 + 64), 0)
+        s = T(lambda: C.moe_route(lg, 8, True))
+        report("  moe route softmax 16384 x 64 top 8", s, 16384 * (64 * 8 + 64), 0)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--only", default="")
@@ -334,6 +404,8 @@ def main():
                 s = T(graph.replay)
             report(f"decode step, 4-layer slice: {label}", s, 0, 0)
             del graph, dec, model
+    if want("latent"):
+        latent_kernels(C, T, report, dev)
     if want("slab"):
         # cost of the adapter k-slab as a function of its width (the k-block is 64 wide whatever R is)
         M, N, K = 24576, 6144, H

@@ -225,7 +225,8 @@ struct LatentDecodeArgs {
 };
 bool latent_decode_tc_supported(const LatentDecodeArgs& a);
 int latent_decode_splits(const LatentDecodeArgs& a, int num_sms);
-const char* latent_decode(const LatentDecodeArgs& a, int n_splits, cudaStream_t s);
+const char* latent_decode_tc(const LatentDecodeArgs& a, int n_splits, int* status, cudaStream_t s);   // csrc/kernels/latent_decode_tc.cu
+const char* latent_decode(const LatentDecodeArgs& a, int n_splits, int* status, cudaStream_t s);
 
 // ---- residual sum + layer norm + depth average (csrc/kernels/post_norm.cu) ----
 struct PostNormArgs {

@@ -1251,7 +1251,7 @@ Tensor latent_decode(const Tensor& q, const Tensor& uk_t, const Tensor& uv, cons
       a.ws = ws.data_ptr<float>();
     }
   }
-  FERRL_CHECK(ferrl::latent_decode(a, n, stream()));
+  FERRL_CHECK(ferrl::latent_decode(a, n, status_word(), stream()));
   Tensor out = out_empty({a.B, a.heads * vdim}, q.options());
   FERRL_CHECK(ferrl::head_gemm(a.dtype, ctx.data_ptr(), static_cast<long long>(a.heads) * a.rank, a.rank, uv.data_ptr(), out.data_ptr(),
                                a.heads * vdim, a.B, a.heads, vdim, a.rank, stream()));

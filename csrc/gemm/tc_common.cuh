@@ -173,15 +173,15 @@ inline bool make_map_2d(CUtensorMap* map, const void* ptr, long long rows, long 
              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-// 3-D form for one head of a packed [rows, heads, cols] operand: head and row strides in elements (multiples of 8),
-// box = [box_rows, 1 head, 64 columns]; columns past `cols` read as zeros although the next head's follow in memory.
+// 3-D form for a [rows, heads, cols] operand: head and row strides in elements (multiples of 8), box = [box_rows,
+// box_heads, 64 columns]; columns past `cols` read as zeros although the next head's follow in memory.
 inline bool make_map_3d(CUtensorMap* map, const void* ptr, long long rows, long long heads, long long cols, long long head_ld,
-                        long long ld, int box_rows) {
+                        long long ld, int box_rows, int box_heads = 1) {
   EncodeTiledFn enc = encode_tiled();
   if (!enc) return false;
   cuuint64_t dims[3] = {static_cast<cuuint64_t>(cols), static_cast<cuuint64_t>(heads), static_cast<cuuint64_t>(rows)};
   cuuint64_t strides[2] = {static_cast<cuuint64_t>(head_ld) * 2, static_cast<cuuint64_t>(ld) * 2};
-  cuuint32_t box[3] = {64u, 1u, static_cast<cuuint32_t>(box_rows)};
+  cuuint32_t box[3] = {64u, static_cast<cuuint32_t>(box_heads), static_cast<cuuint32_t>(box_rows)};
   cuuint32_t estr[3] = {1, 1, 1};
   return enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), dims, strides, box, estr,
              CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,

@@ -6,9 +6,8 @@
 //                           (flash_tc.cu holds the tcgen05 form for bf16)
 //   head_gemm_kernel        out[b, h, :] = W[h] x[b, h, :], one small matrix per head (query absorption, value
 //                           expansion of a decode step) on mma.sync; head_gemm_any_kernel for other types and sizes
-//   latent_decode_kernel    one query per row against the row's cached latents: all heads of a CTA share one pass over
-//                           the cache (mma.sync, cp.async double buffer, split over keys + combine)
-//   latent_decode_any_kernel  the same for any type and size
+//   latent_decode_any_kernel  one query per row against the row's cached latents, any type and size
+//                           (latent_decode_tc.cu holds the tcgen05 form for bf16); latent_combine_kernel joins key ranges
 //
 // Scores, softmax and sink are fp32.  A sink adds exp(sink_h) to the softmax denominator of head h.
 #include <cuda_bf16.h>
@@ -162,32 +161,45 @@ __global__ void head_gemm_any_kernel(const T* __restrict__ x, long long ldx, int
   }
 }
 
-// 64 rows x 64 columns per CTA, k in steps of 64 through a two-stage cp.async ring; K % 8 == 0
+// 64 rows x 64 columns per CTA, k in steps of 64 through a four-stage cp.async ring; K % 8 == 0.  The matrices are
+// weights, so the first stages of w are requested before the wait for the predecessor that writes x.
 constexpr int kHgStage = 2 * 64 * 128;     // bytes: x tile + w tile
+constexpr int kHgDepth = 4;
 __global__ void __launch_bounds__(128) head_gemm_kernel(const bf16* __restrict__ x, long long ldx, int xh,
                                                         const bf16* __restrict__ w, bf16* __restrict__ out,
                                                         long long ldo, int B, int N, int K) {
   using namespace mmah;
   pdl_trigger();
-  pdl_wait();
-  __shared__ __align__(1024) uint8_t smem[2 * kHgStage];
+  extern __shared__ __align__(1024) uint8_t hg_smem[];
   const int n0 = blockIdx.x * 64, b0 = blockIdx.y * 64, h = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int wm = warp & 1, wn = warp >> 1;
   const bf16* xb = x + static_cast<long long>(h) * xh;
   const bf16* wb = w + static_cast<long long>(h) * N * K;
-  const uint32_t base = smem_addr(smem);
+  const uint32_t base = smem_addr(hg_smem);
   const int nk = (K + 63) / 64;
-  auto load = [&](int kt) {
-    const uint32_t s = base + (kt & 1) * kHgStage;
+  auto load_w = [&](int kt) {
+    const uint32_t s = base + (kt % kHgDepth) * kHgStage + 64 * 128;
     for (int i = threadIdx.x; i < 64 * 8; i += 128) {
       const int r = i >> 3, c = i & 7, k = kt * 64 + c * 8;
-      const bool okx = b0 + r < B && k < K, okw = n0 + r < N && k < K;
-      cp_async16(s + sw_off<128>(r, c), okx ? xb + (b0 + r) * ldx + k : xb, okx);
-      cp_async16(s + 64 * 128 + sw_off<128>(r, c), okw ? wb + static_cast<long long>(n0 + r) * K + k : wb, okw);
+      const bool ok = kt < nk && n0 + r < N && k < K;
+      cp_async16(s + sw_off<128>(r, c), ok ? wb + static_cast<long long>(n0 + r) * K + k : wb, ok);
+    }
+  };
+  auto load_x = [&](int kt) {
+    const uint32_t s = base + (kt % kHgDepth) * kHgStage;
+    for (int i = threadIdx.x; i < 64 * 8; i += 128) {
+      const int r = i >> 3, c = i & 7, k = kt * 64 + c * 8;
+      const bool ok = kt < nk && b0 + r < B && k < K;
+      cp_async16(s + sw_off<128>(r, c), ok ? xb + (b0 + r) * ldx + k : xb, ok);
     }
     cp_commit();
   };
+#pragma unroll
+  for (int kt = 0; kt < kHgDepth - 1; ++kt) load_w(kt);
+  pdl_wait();
+#pragma unroll
+  for (int kt = 0; kt < kHgDepth - 1; ++kt) load_x(kt);
   float acc[2][4][4];
 #pragma unroll
   for (int i = 0; i < 2; ++i)
@@ -195,16 +207,12 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(const bf16* __restrict__
     for (int j = 0; j < 4; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.f;
-  load(0);
   for (int kt = 0; kt < nk; ++kt) {
-    if (kt + 1 < nk) {
-      load(kt + 1);
-      cp_wait<1>();
-    } else {
-      cp_wait<0>();
-    }
-    __syncthreads();
-    const uint32_t s = base + (kt & 1) * kHgStage;
+    cp_wait<kHgDepth - 2>();                 // one group a stage, empty ones included: stage kt has landed
+    __syncthreads();                         // and everyone is done with the stage that is loaded next
+    load_w(kt + kHgDepth - 1);
+    load_x(kt + kHgDepth - 1);
+    const uint32_t s = base + (kt % kHgDepth) * kHgStage;
 #pragma unroll
     for (int ks = 0; ks < 4; ++ks) {
       uint32_t a[2][4], bb[2][4];
@@ -220,18 +228,25 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(const bf16* __restrict__
 #pragma unroll
         for (int j = 0; j < 4; ++j) mma16816(acc[i][j], a[i], bb[j >> 1][(j & 1) * 2], bb[j >> 1][(j & 1) * 2 + 1]);
     }
-    __syncthreads();
   }
+  cp_wait<0>();
   bf16* ob = out + static_cast<long long>(h) * N;
+  const bool pairs = (N % 2) == 0 && (ldo % 2) == 0;
 #pragma unroll
   for (int i = 0; i < 2; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
+      for (int e = 0; e < 4; e += 2) {
         const int r = b0 + wm * 32 + i * 16 + (lane >> 2) + (e >> 1) * 8;
-        const int c = n0 + wn * 32 + j * 8 + (lane & 3) * 2 + (e & 1);
-        if (r < B && c < N) ob[r * ldo + c] = __float2bfloat16_rn(acc[i][j][e]);
+        const int c = n0 + wn * 32 + j * 8 + (lane & 3) * 2;
+        if (r >= B || c >= N) continue;
+        if (pairs) {
+          *reinterpret_cast<uint32_t*>(ob + r * ldo + c) = pack_bf16(acc[i][j][e], acc[i][j][e + 1]);
+        } else {
+          ob[r * ldo + c] = __float2bfloat16_rn(acc[i][j][e]);
+          if (c + 1 < N) ob[r * ldo + c + 1] = __float2bfloat16_rn(acc[i][j][e + 1]);
+        }
       }
 }
 
@@ -284,254 +299,7 @@ __global__ void __launch_bounds__(128) latent_decode_any_kernel(LatentDecodeArgs
   for (int c = threadIdx.x; c < a.rank; c += 128) o[c] = from_f<T>(so[c] * inv);
 }
 
-// ------------------------------------------------------------------------------------------------ decode, tensor cores
-// A CTA owns 16 * MT heads of one row and a range of its cached latents.  Key tiles of 64 rows go through a two-stage
-// cp.async ring; a shared-memory row holds [latent, zero-padded to NT * 64 | rotated part, zero-padded to 16s].
-// Scores: warp (m, n) covers one 16-head tile and 64 / (8 / MT) keys; the context: warp w covers NT n8-tiles of the
-// latent for all heads, B fragments by transposed ldmatrix of the same tile.
-constexpr int kLdKeys = 64;
-
-__device__ __forceinline__ uint32_t ld_off(int row, int chunk, int pitch) {
-  return static_cast<uint32_t>(row * pitch + ((chunk ^ (row & 7)) << 4));
-}
-
-template <int NT, int MT>
-__global__ void __launch_bounds__(256, 1) latent_decode_kernel(LatentDecodeArgs a, int n_splits, int pitch) {
-  using namespace mmah;
-  constexpr int HB = 16 * MT, NW = 8 / MT, NK8 = kLdKeys / NW / 8;   // NK8 n8-tiles of keys per score warp
-  extern __shared__ __align__(1024) uint8_t smem[];
-  const int KP = NT * 64, ks_total = KP / 16 + (a.rot + 15) / 16;
-  uint8_t* sQ = smem;
-  uint8_t* sK = sQ + HB * pitch;
-  bf16* sP = reinterpret_cast<bf16*>(sK + 2 * kLdKeys * pitch);      // [HB][64], chunk-swizzled rows of 128 bytes
-  float* s_max = reinterpret_cast<float*>(sP + HB * kLdKeys);        // [HB][NW]
-  float* s_m = s_max + HB * NW;                                      // [HB] running maximum (score * scale * log2e)
-  float* s_corr = s_m + HB;                                          // [HB]
-  float* s_l = s_corr + HB;                                          // [HB][NW]
-  pdl_trigger();
-  pdl_wait();
-  const int split = blockIdx.x, hb = blockIdx.y * HB, b = blockIdx.z;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int n = min(max(a.count[b], 0), a.slots);
-  const int tiles = (n + kLdKeys - 1) / kLdKeys;
-  const int t_lo = static_cast<int>(static_cast<long long>(tiles) * split / n_splits);
-  const int t_hi = static_cast<int>(static_cast<long long>(tiles) * (split + 1) / n_splits);
-  const bf16* cache = static_cast<const bf16*>(a.cache) + static_cast<long long>(b) * a.slots * a.width;
-  const uint32_t q_base = smem_addr(sQ), k_base = smem_addr(sK), p_base = smem_addr(sP);
-  const int kc = KP / 8, kc_valid = a.rank / 8, rc = a.rot / 8;
-  const int chunks = ks_total * 2;                                   // 16-byte chunks per row that the MMAs read
-  auto load_keys = [&](int t) {
-    const uint32_t s = k_base + ((t - t_lo) & 1) * kLdKeys * pitch;
-    for (int i = threadIdx.x; i < kLdKeys * chunks; i += 256) {
-      const int r = i / chunks, c = i - r * chunks, key = t * kLdKeys + r;
-      int src = c;
-      bool ok = key < n;
-      if (c < kc) {
-        ok = ok && c < kc_valid;
-      } else {
-        src = kc_valid + c - kc;
-        ok = ok && c - kc < rc;
-      }
-      cp_async16(s + ld_off(r, c, pitch), ok ? cache + static_cast<long long>(key) * a.width + src * 8 : cache, ok);
-    }
-    cp_commit();
-  };
-  {
-    const bf16* qa = static_cast<const bf16*>(a.qa) + (static_cast<long long>(b) * a.heads) * a.rank;
-    const bf16* qr = static_cast<const bf16*>(a.qr) + b * a.ld_qr;
-    for (int i = threadIdx.x; i < HB * chunks; i += 256) {
-      const int r = i / chunks, c = i - r * chunks, h = hb + r;
-      const bf16* src = qa;
-      bool ok = h < a.heads;
-      if (c < kc) {
-        ok = ok && c < kc_valid;
-        if (ok) src = qa + static_cast<long long>(h) * a.rank + c * 8;
-      } else {
-        ok = ok && c - kc < rc;
-        if (ok) src = qr + static_cast<long long>(h) * a.qr_hs + (c - kc) * 8;
-      }
-      cp_async16(q_base + ld_off(r, c, pitch), src, ok);
-    }
-    cp_commit();
-  }
-  for (int i = threadIdx.x; i < HB; i += 256) s_m[i] = -INFINITY;
-  float o[MT][NT][4];
-#pragma unroll
-  for (int i = 0; i < MT; ++i)
-#pragma unroll
-    for (int j = 0; j < NT; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) o[i][j][e] = 0.f;
-  float l_part[2] = {0.f, 0.f};
-  const int wm = warp / NW, wn = warp % NW;                          // score role
-  const int r_lo = wm * 16 + (lane >> 2);                            // this lane's head rows: r_lo, r_lo + 8
-  const float c2 = a.scale * kLog2e;
-  if (t_lo < t_hi) load_keys(t_lo);
-  for (int t = t_lo; t < t_hi; ++t) {
-    cp_wait<0>();
-    __syncthreads();                                                 // tile t is here; everyone is done with tile t - 1
-    if (t + 1 < t_hi) load_keys(t + 1);
-    const uint32_t ks = k_base + ((t - t_lo) & 1) * kLdKeys * pitch;
-    float s[NK8][4];
-#pragma unroll
-    for (int j = 0; j < NK8; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) s[j][e] = 0.f;
-#pragma unroll 4
-    for (int k = 0; k < ks_total; ++k) {
-      uint32_t av[4];
-      ldsm4(q_base + ld_off(wm * 16 + (lane & 15), k * 2 + (lane >> 4), pitch), av[0], av[1], av[2], av[3]);
-      if (NK8 == 1) {
-        // one 8-key tile: lanes 0-15 address it, the other two matrices repeat it
-        uint32_t b0, b1, b2, b3;
-        ldsm4(ks + ld_off(wn * 8 + (lane & 7), k * 2 + ((lane >> 3) & 1), pitch), b0, b1, b2, b3);
-        mma16816(s[0], av, b0, b1);
-      } else {
-#pragma unroll
-        for (int j = 0; j < NK8; j += 2) {
-          uint32_t b0, b1, b2, b3;
-          ldsm4(ks + ld_off((wn * NK8 + j) * 8 + (lane & 7) + ((lane >> 4) << 3), k * 2 + ((lane >> 3) & 1), pitch), b0, b1, b2, b3);
-          mma16816(s[j], av, b0, b1);
-          mma16816(s[j + 1], av, b2, b3);
-        }
-      }
-    }
-    // scaled scores, keys past the end masked; row maxima over this warp's keys, then over the score warps
-    float mx[2] = {-INFINITY, -INFINITY};
-#pragma unroll
-    for (int j = 0; j < NK8; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int key = t * kLdKeys + (wn * NK8 + j) * 8 + (lane & 3) * 2 + (e & 1);
-        s[j][e] = key < n ? s[j][e] * c2 : -INFINITY;
-        mx[e >> 1] = fmaxf(mx[e >> 1], s[j][e]);
-      }
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));
-      mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 2));
-      if ((lane & 3) == 0) s_max[(r_lo + i * 8) * NW + wn] = mx[i];
-    }
-    __syncthreads();
-    float m_new[2], corr[2];
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const float m_old = s_m[r_lo + i * 8];
-      float v = m_old;
-#pragma unroll
-      for (int w = 0; w < NW; ++w) v = fmaxf(v, s_max[(r_lo + i * 8) * NW + w]);
-      m_new[i] = v;                                                  // finite: a tile holds at least one key
-      corr[i] = m_old == -INFINITY ? 0.f : exp2f(m_old - v);
-      l_part[i] *= corr[i];
-    }
-#pragma unroll
-    for (int j = 0; j < NK8; ++j) {
-      float p[4];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        p[e] = s[j][e] == -INFINITY ? 0.f : exp2f(s[j][e] - m_new[e >> 1]);
-        l_part[e >> 1] += p[e];
-      }
-      const int c = (wn * NK8 + j);                                  // 8-key chunk of the P row
-#pragma unroll
-      for (int i = 0; i < 2; ++i)
-        *reinterpret_cast<uint32_t*>(reinterpret_cast<uint8_t*>(sP) + ld_off(r_lo + i * 8, c, 128) + (lane & 3) * 4) =
-            pack_bf16(p[2 * i], p[2 * i + 1]);
-    }
-    if (wn == 0 && (lane & 3) == 0) {
-#pragma unroll
-      for (int i = 0; i < 2; ++i) s_corr[r_lo + i * 8] = corr[i];
-    }
-    __syncthreads();
-    if (wn == 0 && (lane & 3) == 0) {
-#pragma unroll
-      for (int i = 0; i < 2; ++i) s_m[r_lo + i * 8] = m_new[i];      // read again only after the next two barriers
-    }
-    // context: o = o * corr + P C
-#pragma unroll
-    for (int i = 0; i < MT; ++i) {
-      const float f0 = s_corr[i * 16 + (lane >> 2)], f1 = s_corr[i * 16 + (lane >> 2) + 8];
-#pragma unroll
-      for (int j = 0; j < NT; ++j) {
-        o[i][j][0] *= f0;
-        o[i][j][1] *= f0;
-        o[i][j][2] *= f1;
-        o[i][j][3] *= f1;
-      }
-    }
-#pragma unroll
-    for (int k = 0; k < kLdKeys / 16; ++k) {
-      uint32_t av[MT][4];
-#pragma unroll
-      for (int i = 0; i < MT; ++i)
-        ldsm4(p_base + ld_off(i * 16 + (lane & 15), k * 2 + (lane >> 4), 128), av[i][0], av[i][1], av[i][2], av[i][3]);
-      if (NT == 1) {
-        uint32_t b0, b1, b2, b3;
-        ldsm4t(ks + ld_off(k * 16 + (lane & 15), warp, pitch), b0, b1, b2, b3);
-#pragma unroll
-        for (int i = 0; i < MT; ++i) mma16816(o[i][0], av[i], b0, b1);
-      } else {
-#pragma unroll
-        for (int j = 0; j + 1 < NT; j += 2) {
-          uint32_t b0, b1, b2, b3;
-          ldsm4t(ks + ld_off(k * 16 + (lane & 15), warp * NT + j + (lane >> 4), pitch), b0, b1, b2, b3);
-#pragma unroll
-          for (int i = 0; i < MT; ++i) {
-            mma16816(o[i][j], av[i], b0, b1);
-            mma16816(o[i][j + 1], av[i], b2, b3);
-          }
-        }
-        if (NT & 1) {
-          uint32_t b0, b1, b2, b3;
-          ldsm4t(ks + ld_off(k * 16 + (lane & 15), warp * NT + NT - 1, pitch), b0, b1, b2, b3);
-#pragma unroll
-          for (int i = 0; i < MT; ++i) mma16816(o[i][NT - 1], av[i], b0, b1);
-        }
-      }
-    }
-  }
-  cp_wait<0>();
-  // row sums over the lanes and warps of each head
-#pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    l_part[i] += __shfl_xor_sync(0xffffffffu, l_part[i], 1);
-    l_part[i] += __shfl_xor_sync(0xffffffffu, l_part[i], 2);
-    if ((lane & 3) == 0) s_l[(r_lo + i * 8) * NW + wn] = l_part[i];
-  }
-  __syncthreads();
-#pragma unroll
-  for (int i = 0; i < MT; ++i)
-#pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int r = i * 16 + (lane >> 2) + half * 8, h = hb + r;
-      if (h >= a.heads) continue;
-      float l = 0.f;
-#pragma unroll
-      for (int w = 0; w < NW; ++w) l += s_l[r * NW + w];
-      const float m = s_m[r];
-      const long long oh = static_cast<long long>(b) * a.heads + h;
-      if (n_splits == 1) {
-        float inv = 0.f;
-        if (n > 0) inv = 1.f / (a.sink ? l + exp2f(a.sink[h] * kLog2e - m) : l);
-        bf16* dst = static_cast<bf16*>(a.ctx) + oh * a.rank;
-#pragma unroll
-        for (int j = 0; j < NT; ++j) {
-          const int c = (warp * NT + j) * 8 + (lane & 3) * 2;
-          if (c < a.rank)
-            *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16(o[i][j][half * 2] * inv, o[i][j][half * 2 + 1] * inv);
-        }
-      } else {
-        float* dst = a.ws + (oh * n_splits + split) * (a.rank + 2);
-#pragma unroll
-        for (int j = 0; j < NT; ++j) {
-          const int c = (warp * NT + j) * 8 + (lane & 3) * 2;
-          if (c < a.rank) *reinterpret_cast<float2*>(dst + c) = make_float2(o[i][j][half * 2], o[i][j][half * 2 + 1]);
-        }
-        if (warp == 0 && (lane & 3) == 0) *reinterpret_cast<float2*>(dst + a.rank) = make_float2(m, l);
-      }
-    }
-}
-
+// ------------------------------------------------------------------------------------------------ key ranges of a row
 __global__ void latent_combine_kernel(const float* __restrict__ ws, const float* __restrict__ sink, bf16* __restrict__ ctx,
                                       int heads, int rank, int n_splits) {
   pdl_trigger();
@@ -554,41 +322,6 @@ __global__ void latent_combine_kernel(const float* __restrict__ ws, const float*
       if (q[rank] != -INFINITY) o += q[c] * exp2f(q[rank] - m);
     }
     ctx[oh * rank + c] = __float2bfloat16_rn(o * inv);
-  }
-}
-
-int decode_pitch(const LatentDecodeArgs& a) {
-  const int kp = (a.rank + 63) / 64 * 64, rp = (a.rot + 15) / 16 * 16;
-  return (kp + rp + 63) / 64 * 128;
-}
-size_t decode_smem(int HB, int NW, int pitch) {
-  return static_cast<size_t>(HB) * pitch + 2 * kLdKeys * static_cast<size_t>(pitch) + HB * kLdKeys * 2 +
-         static_cast<size_t>(HB) * (2 * NW + 2) * 4;
-}
-
-template <int NT, int MT>
-const char* launch_decode(const LatentDecodeArgs& a, int n_splits, cudaStream_t s) {
-  const int pitch = decode_pitch(a);
-  const size_t smem = decode_smem(16 * MT, 8 / MT, pitch);
-  auto kern = latent_decode_kernel<NT, MT>;
-  // the largest request of this instance: rotated parts of up to 128 entries
-  if (!FERRL_ONCE_PER_DEVICE(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) == cudaSuccess))
-    return "latent_decode: cannot reserve shared memory";
-  launch_pdl(kern, dim3(n_splits, (a.heads + 16 * MT - 1) / (16 * MT), a.B), dim3(256), smem, s, a, n_splits, pitch);
-  count_launch();
-  return nullptr;
-}
-template <int MT>
-const char* pick_decode(const LatentDecodeArgs& a, int n_splits, cudaStream_t s) {
-  switch ((a.rank + 63) / 64) {
-    case 1: return launch_decode<1, MT>(a, n_splits, s);
-    case 2: return launch_decode<2, MT>(a, n_splits, s);
-    case 3: return launch_decode<3, MT>(a, n_splits, s);
-    case 4: return launch_decode<4, MT>(a, n_splits, s);
-    case 5: return launch_decode<5, MT>(a, n_splits, s);
-    case 6: return launch_decode<6, MT>(a, n_splits, s);
-    case 7: return launch_decode<7, MT>(a, n_splits, s);
-    default: return launch_decode<8, MT>(a, n_splits, s);
   }
 }
 
@@ -625,7 +358,9 @@ const char* head_gemm(int dtype, const void* x, long long ldx, int xh, const voi
                       int N, int K, cudaStream_t s) {
   if (B == 0) return nullptr;
   if (dtype == kBF16 && K % 8 == 0 && ldx % 8 == 0 && xh % 8 == 0 && al16(x) && al16(w)) {
-    launch_pdl(head_gemm_kernel, dim3((N + 63) / 64, (B + 63) / 64, H), dim3(128), 0, s, static_cast<const bf16*>(x), ldx, xh,
+    if (!FERRL_ONCE_PER_DEVICE(cudaFuncSetAttribute(head_gemm_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kHgDepth * kHgStage) == cudaSuccess))
+      return "head_gemm: cannot reserve shared memory";
+    launch_pdl(head_gemm_kernel, dim3((N + 63) / 64, (B + 63) / 64, H), dim3(128), kHgDepth * kHgStage, s, static_cast<const bf16*>(x), ldx, xh,
                static_cast<const bf16*>(w), static_cast<bf16*>(out), ldo, B, N, K);
   } else {
     const dim3 grid(std::min((N + 7) / 8, 64), H, B);
@@ -640,19 +375,7 @@ const char* head_gemm(int dtype, const void* x, long long ldx, int xh, const voi
   return cudaGetLastError() == cudaSuccess ? nullptr : "head_gemm launch failed";
 }
 
-bool latent_decode_tc_supported(const LatentDecodeArgs& a) {
-  return a.dtype == kBF16 && a.rank % 8 == 0 && a.rank <= 512 && a.rot % 8 == 0 && a.rot <= 128 && a.width % 8 == 0 &&
-         a.ld_qr % 8 == 0 && a.qr_hs % 8 == 0 && al16(a.qa) && al16(a.qr) && al16(a.cache) &&
-         decode_smem(a.heads > 16 ? 32 : 16, a.heads > 16 ? 4 : 8, decode_pitch(a)) <= 227 * 1024;
-}
-
-// key ranges per row: enough CTAs for the device, at least two key tiles each
-int latent_decode_splits(const LatentDecodeArgs& a, int num_sms) {
-  const int ctas = a.B * ((a.heads + 31) / 32), tiles = (a.slots + kLdKeys - 1) / kLdKeys;
-  return std::max(1, std::min({num_sms / std::max(ctas, 1), tiles / 2, 64}));
-}
-
-const char* latent_decode(const LatentDecodeArgs& a, int n_splits, cudaStream_t s) {
+const char* latent_decode(const LatentDecodeArgs& a, int n_splits, int* status, cudaStream_t s) {
   if (a.B == 0) return nullptr;
   if (!latent_decode_tc_supported(a)) {
     const size_t smem = static_cast<size_t>(2 * a.rank + a.rot) * 4;
@@ -668,8 +391,7 @@ const char* latent_decode(const LatentDecodeArgs& a, int n_splits, cudaStream_t 
     return cudaGetLastError() == cudaSuccess ? nullptr : "latent_decode launch failed";
   }
   if (n_splits > 1 && !a.ws) return "latent_decode: workspace missing";
-  const char* err = a.heads > 16 ? pick_decode<2>(a, n_splits, s) : pick_decode<1>(a, n_splits, s);
-  if (err) return err;
+  if (const char* err = latent_decode_tc(a, n_splits, status, s)) return err;
   if (n_splits > 1) {
     launch_pdl(latent_combine_kernel, dim3(a.B * a.heads), dim3(128), 0, s, static_cast<const float*>(a.ws), a.sink,
                static_cast<bf16*>(a.ctx), a.heads, a.rank, n_splits);

@@ -570,7 +570,7 @@ def post_norm(x, y, weight, bias, eps, alpha, gate, gate_bias, history, coef, ca
     def native_fn(x_, y_, w_, b_, g_, gb_, h_, c_):
         W = x_.shape[-1]
         nxt, low, r = lib().post_norm(x_.contiguous(), None if y_ is None else _rows2(y_, W), None if g_ is None else _rows2(g_, W),
-                                      gb_, w_, b_, float(eps), float(alpha), h_, c_, cast == torch.bfloat16, out)
+                                      gb_, w_, b_, float(eps), float(alpha), h_, c_, cast == torch.bfloat16 or _bf16(y_), out)
         return nxt, low, r
     args = (x, y, weight, bias, gate, gate_bias, history, coef)
     if _wants_grad(*args):

@@ -40,7 +40,7 @@ ONE = config(40, 32, [(mixer(1, 8, 8, 16, 8, window=500), moe(1, 1, 16))], alpha
 # sizes for the tensor-core kernels: whole 64-column atoms, more than 16 heads, wide latents
 WIDE = config(160, 128, [
     (mixer(20, 64, 32, 64, 128, window=70), dense(128)),
-    (mixer(4, 128, 64, 128, 192, window=130), moe(6, 2, 64)),
+    (mixer(4, 128, 64, 128, 192, window=130), moe(3, 3, 64)),
     (mixer(2, 96, 16, 136, 72, window=17), None),
 ], alpha=1.2)
 CASES = {"mixed": MIXED, "odd": ODD, "one": ONE, "wide": WIDE}

@@ -1,7 +1,7 @@
 """Per-kernel timings at the headline model's shapes, against the measured roofline.
 
     python bench_kernels.py [--only gemm,attn,...] [--iters 20] [--json out.json]
-    python bench_kernels.py --profile-case gemm|gemm_2cta_256|gemm_lora|gemm_decode|decode_attn|sample|flash|flash_tc1|flash_tc2|flash_bwd|rmsnorm|swiglu|qk_norm_rope|logprob|lora_grad|moe_grouped|gdn_decode|gdn_chunk|gdn_tc_fwd|gdn_tc_bwd|flash_tc3_d256|flash_tc3_window|decode_attn_group|logprob_head   # small, for a profiler
+    python bench_kernels.py --profile-case gemm|gemm_2cta_256|gemm_lora|gemm_decode|decode_attn|sample|flash|flash_tc1|flash_tc2|flash_bwd|rmsnorm|swiglu|qk_norm_rope|logprob|lora_grad|moe_grouped|gdn_decode|gdn_chunk|gdn_tc_fwd|gdn_tc_bwd|flash_tc3_d256|flash_tc3_window|decode_attn_group|logprob_head|latent_decode|latent_prefill|post_norm   # small, for a profiler
 
 Every kernel is timed with CUDA events on the launching stream after warm-up, with a buffer
 larger than L2 written between iterations (cold L2), and reported as achieved bytes/s or FLOP/s
@@ -179,6 +179,17 @@ def profile_case(name, C):
     elif name == "flash_tc1":
         q, k, v = rnd(8, 1536, 32, 128), rnd(8, 1536, 8, 128), rnd(8, 1536, 8, 128)
         fn = lambda: C.attention(q, k, v, scale=128 ** -0.5, causal=True, variant=2)
+    elif name == "latent_decode":
+        q, uk, uv, cache = rnd(128, 32, 192), rnd(32, 512, 128), rnd(32, 128, 512), rnd(128, 2048, 576)
+        cnt = torch.full((128,), 2048, device=dev, dtype=torch.int32)
+        fn = lambda: C.latent_decode(q, uk, uv, cache, cnt, rank=512, scale=0.07)
+    elif name == "latent_prefill":
+        q, kv, lat = rnd(8, 2048, 32, 192), rnd(8, 2048, 32 * 256), rnd(8, 2048, 576)
+        fn = lambda: C.latent_attention(q, kv, lat, dim=128, vdim=128, rank=512, scale=0.07, window=1024)
+    elif name == "post_norm":
+        x, y, gt = torch.randn(8192, 4096, device=dev), rnd(8192, 4096), rnd(8192, 4096)
+        v1, hist, coef = torch.ones(4096, device=dev), torch.randn(2, 8192, 4096, device=dev), torch.ones(3, device=dev)
+        fn = lambda: C.post_norm(x, y, v1, v1, 1e-6, 2.0, gt, v1, hist, coef, bf, None)
     else:
         raise SystemExit(f"unknown profile case {name!r}")
     evs = []

@@ -161,10 +161,10 @@ __global__ void head_gemm_any_kernel(const T* __restrict__ x, long long ldx, int
   }
 }
 
-// 64 rows x 64 columns per CTA, k in steps of 64 through a four-stage cp.async ring; K % 8 == 0.  The matrices are
+// 64 rows x 64 columns per CTA, k in steps of 64 through a DEPTH-stage cp.async ring; K % 8 == 0.  The matrices are
 // weights, so the first stages of w are requested before the wait for the predecessor that writes x.
 constexpr int kHgStage = 2 * 64 * 128;     // bytes: x tile + w tile
-constexpr int kHgDepth = 4;
+template <int DEPTH>
 __global__ void __launch_bounds__(128) head_gemm_kernel(const bf16* __restrict__ x, long long ldx, int xh,
                                                         const bf16* __restrict__ w, bf16* __restrict__ out,
                                                         long long ldo, int B, int N, int K) {
@@ -179,27 +179,28 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(const bf16* __restrict__
   const uint32_t base = smem_addr(hg_smem);
   const int nk = (K + 63) / 64;
   auto load_w = [&](int kt) {
-    const uint32_t s = base + (kt % kHgDepth) * kHgStage + 64 * 128;
+    if (kt >= nk) return;
+    const uint32_t s = base + (kt % DEPTH) * kHgStage + 64 * 128;
     for (int i = threadIdx.x; i < 64 * 8; i += 128) {
       const int r = i >> 3, c = i & 7, k = kt * 64 + c * 8;
-      const bool ok = kt < nk && n0 + r < N && k < K;
+      const bool ok = n0 + r < N && k < K;
       cp_async16(s + sw_off<128>(r, c), ok ? wb + static_cast<long long>(n0 + r) * K + k : wb, ok);
     }
   };
-  auto load_x = [&](int kt) {
-    const uint32_t s = base + (kt % kHgDepth) * kHgStage;
-    for (int i = threadIdx.x; i < 64 * 8; i += 128) {
+  auto load_x = [&](int kt) {               // closes the stage's copy group (an empty one past the end)
+    const uint32_t s = base + (kt % DEPTH) * kHgStage;
+    for (int i = threadIdx.x; kt < nk && i < 64 * 8; i += 128) {
       const int r = i >> 3, c = i & 7, k = kt * 64 + c * 8;
-      const bool ok = kt < nk && b0 + r < B && k < K;
+      const bool ok = b0 + r < B && k < K;
       cp_async16(s + sw_off<128>(r, c), ok ? xb + (b0 + r) * ldx + k : xb, ok);
     }
     cp_commit();
   };
 #pragma unroll
-  for (int kt = 0; kt < kHgDepth - 1; ++kt) load_w(kt);
+  for (int kt = 0; kt < DEPTH - 1; ++kt) load_w(kt);
   pdl_wait();
 #pragma unroll
-  for (int kt = 0; kt < kHgDepth - 1; ++kt) load_x(kt);
+  for (int kt = 0; kt < DEPTH - 1; ++kt) load_x(kt);
   float acc[2][4][4];
 #pragma unroll
   for (int i = 0; i < 2; ++i)
@@ -208,11 +209,11 @@ __global__ void __launch_bounds__(128) head_gemm_kernel(const bf16* __restrict__
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[i][j][e] = 0.f;
   for (int kt = 0; kt < nk; ++kt) {
-    cp_wait<kHgDepth - 2>();                 // one group a stage, empty ones included: stage kt has landed
+    cp_wait<DEPTH - 2>();                 // one group a stage, empty ones included: stage kt has landed
     __syncthreads();                         // and everyone is done with the stage that is loaded next
-    load_w(kt + kHgDepth - 1);
-    load_x(kt + kHgDepth - 1);
-    const uint32_t s = base + (kt % kHgDepth) * kHgStage;
+    load_w(kt + DEPTH - 1);
+    load_x(kt + DEPTH - 1);
+    const uint32_t s = base + (kt % DEPTH) * kHgStage;
 #pragma unroll
     for (int ks = 0; ks < 4; ++ks) {
       uint32_t a[2][4], bb[2][4];
@@ -358,10 +359,15 @@ const char* head_gemm(int dtype, const void* x, long long ldx, int xh, const voi
                       int N, int K, cudaStream_t s) {
   if (B == 0) return nullptr;
   if (dtype == kBF16 && K % 8 == 0 && ldx % 8 == 0 && xh % 8 == 0 && al16(x) && al16(w)) {
-    if (!FERRL_ONCE_PER_DEVICE(cudaFuncSetAttribute(head_gemm_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kHgDepth * kHgStage) == cudaSuccess))
+    const bf16 *xp = static_cast<const bf16*>(x), *wp = static_cast<const bf16*>(w);
+    const dim3 grid((N + 63) / 64, (B + 63) / 64, H);
+    // short contractions take three stages (four CTAs an SM), long ones five
+    if (!FERRL_ONCE_PER_DEVICE(
+            cudaFuncSetAttribute(head_gemm_kernel<3>, cudaFuncAttributeMaxDynamicSharedMemorySize, 3 * kHgStage) == cudaSuccess &&
+            cudaFuncSetAttribute(head_gemm_kernel<5>, cudaFuncAttributeMaxDynamicSharedMemorySize, 5 * kHgStage) == cudaSuccess))
       return "head_gemm: cannot reserve shared memory";
-    launch_pdl(head_gemm_kernel, dim3((N + 63) / 64, (B + 63) / 64, H), dim3(128), kHgDepth * kHgStage, s, static_cast<const bf16*>(x), ldx, xh,
-               static_cast<const bf16*>(w), static_cast<bf16*>(out), ldo, B, N, K);
+    if (K <= 128) launch_pdl(head_gemm_kernel<3>, grid, dim3(128), 3 * kHgStage, s, xp, ldx, xh, wp, static_cast<bf16*>(out), ldo, B, N, K);
+    else launch_pdl(head_gemm_kernel<5>, grid, dim3(128), 5 * kHgStage, s, xp, ldx, xh, wp, static_cast<bf16*>(out), ldo, B, N, K);
   } else {
     const dim3 grid(std::min((N + 7) / 8, 64), H, B);
     if (dtype == kF32)

@@ -11,7 +11,9 @@
 namespace ferrl {
 
 enum { kBF16 = 0, kF32 = 1 };
-enum { kActSilu = 0, kActGeluTanh = 1 };
+enum { kActSilu = 0, kActGeluTanh = 1, kActClipped = 2 };
+// gated activation act(gate) * up; kActClipped: g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, +-limit)
+struct GluAct { int act; float alpha, limit; };
 
 // ---- tcgen05 GEMM: out[M,N] = A[M,K] B[N,K]^T (+ A2[M,K2] B2[N,K2]^T) (+ residual) ----
 struct GemmArgs {
@@ -52,7 +54,7 @@ struct GemmArgs {
   // dependency wait (only where B is never written by an earlier kernel of the same stream)
   int pdl;
   // GLU epilogue: B rows interleaved in groups of 16 (8 gate, 8 up); out is [M, N/2]; 1 SiLU, 2 tanh-GELU
-  int glu_act;
+  int glu_act; float glu_alpha, glu_limit;
   // RMSNorm folded around the projection (one-SM and cluster split-k kernels, bf16 output):
   // ss_in [ss_parts, ss_ld] fp32 partial row sums of squares of A's rows (rows are scaled by
   // rsqrt(sum * ss_inv_k + ss_eps) in the epilogue); ss_out [parts, ss_ld] receives the partial row sums
@@ -126,7 +128,7 @@ const char* kv_append(int dtype, const void* k, const void* v, long long ldv, vo
                       int batch, int smax, int HD, cudaStream_t s);
 
 // ---- misc ----
-const char* glu(int dtype, bool backward, const void* gu, const void* dout, void* out, long long rows, int F, int act,
+const char* glu(int dtype, bool backward, const void* gu, const void* dout, void* out, long long rows, int F, GluAct act,
                 cudaStream_t s);
 const char* embedding(int dtype, const long long* ids, const void* table, void* out, long long n_tok, int H,
                       long long vocab, float scale, cudaStream_t s);
@@ -239,6 +241,66 @@ struct PostNormArgs {
   float* r; float* next; void* cast; int cast_dtype;     // outputs, each may be null
 };
 const char* post_norm(const PostNormArgs& a, cudaStream_t s);
+
+// ---- hyper-connections and streams (csrc/kernels/hyper.cu) ----
+struct HyperNormArgs {
+  float* x; long long rows; int W, ns;       // [rows, ns, W]; rewritten in place when y and store are set
+  const void* y; long long ld_y; int y_dtype;   // sublayer output or null
+  const float* mix; const float* out;        // [ns (from), ns (to)], [ns]: coefficients of the sublayer that gave y
+  const float* in;                           // [ns]: what the next sublayer reads; null: the plain sum
+  const float* w; float eps, scale;          // norm weight around zero [W]; factor on the result
+  void* h; int h_dtype; int store;
+};
+const char* hyper_norm(const HyperNormArgs& a, cudaStream_t s);
+// out[t, s, :] = table[ids[t]] + pe[position], position kv_len[t] or pos[t % S]
+const char* embed_streams(int dtype, const long long* ids, const void* table, const float* pe, const long long* pos, const int* kv_len,
+                          long long S, float* out, long long n_tok, int W, int ns, long long vocab, long long max_pos, cudaStream_t s);
+
+// ---- state-space duality layers (csrc/kernels/ssm.cu) ----
+const char* ssm_conv(int dtype, const void* x, long long x_bs, long long x_ts, const float* w, const float* bias, void* y, int B, int L, int C,
+                     int K, cudaStream_t s);
+struct SsmScanArgs {
+  int dtype;
+  const void* x; const void* Bm; const void* Cm; long long bs, ts;   // [B, T, H*P], [B, T, G*N] x 2: one batch and token stride
+  const void* dt; long long dt_bs, dt_ts;                            // raw step sizes [B, T, H]
+  const float* dt_bias; const float* A_log; const float* D;          // [H]
+  const long long* lens;                                             // [B] or null: tokens that count
+  void* y; float* state;                                             // [B, T, H*P]; [B, H, N, P] or null
+  int B, T, H, P, N, G;
+};
+const char* ssm_scan(const SsmScanArgs& a, cudaStream_t s);
+struct SsmStepArgs {
+  int dtype;
+  const void* x; long long ld_x;                   // this token's convolution inputs [B, C], C = H*P + 2*G*N
+  const void* dt; long long ld_dt;                 // raw step sizes [B, H]
+  const float* conv_w; const float* conv_b;        // [C, K], [C] or null
+  const float* dt_bias; const float* A_log; const float* D;
+  void* ring; float* state;                        // [B, K, C] inputs by position % K; [B, H, N, P]
+  const int* kv_len; const unsigned char* active;  // positions; null or 0 for rows that do not move
+  void* y; int B, H, P, N, G, K, C;
+};
+const char* ssm_step(const SsmStepArgs& a, cudaStream_t s);
+const char* gated_group_norm(int dtype, const void* y, long long ld_y, const void* z, long long ld_z, const float* w, void* out, long long rows,
+                             int W, int groups, float eps, cudaStream_t s);
+
+// ---- distance-biased sliding-window attention, values = keys (csrc/kernels/bias_attn.cu) ----
+struct BiasFwdArgs {
+  int dtype;
+  const void* q; const void* k; void* out;         // [B, S, Hq, D], [B, S, Hkv, D], [B, S, Hq*D] contiguous
+  long long q_bs, q_ts, k_bs, k_ts;
+  const float* bias; long long bias_ld;            // [Hq, bias_ld], at least min(window, S) distances
+  int B, S, Hq, Hkv, D, window; float scale;
+};
+const char* bias_fwd_any(const BiasFwdArgs& a, cudaStream_t s);
+struct BiasDecodeArgs {
+  int dtype;
+  const void* q; long long ld_q; const void* k; long long ld_k;   // this token's [B, Hq*D] and [B, Hkv*D]
+  void* cache; int slots;                          // [B, slots, Hkv*D], a ring by position % slots
+  const int* kv_len; const unsigned char* active;
+  const float* bias; long long bias_ld; void* out; // [B, Hq*D]
+  int B, Hq, Hkv, D; float scale;
+};
+const char* bias_decode_any(const BiasDecodeArgs& a, cudaStream_t s);
 
 // ---- flash attention (prefill / training) ----
 struct FlashArgs {

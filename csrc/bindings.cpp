@@ -283,12 +283,12 @@ Tensor gemm(const Tensor& A, const Tensor& B, const optional<Tensor>& A2, const 
 
 // act(x Wg^T) * (x Wu^T) in one kernel: W holds the gate and up rows interleaved in groups of 16
 // (8 gate rows, then the 8 up rows of the same features); returns [M, N/2].
-Tensor gemm_glu(const Tensor& A, const Tensor& B, int64_t act, bool static_b) {
+Tensor gemm_glu(const Tensor& A, const Tensor& B, int64_t act, bool static_b, double alpha, double limit) {
   TORCH_CHECK(A.is_cuda() && B.is_cuda() && A.scalar_type() == at::kBFloat16 && B.scalar_type() == at::kBFloat16 &&
                   A.dim() == 2 && B.dim() == 2 && A.size(1) == B.size(1) && A.stride(1) == 1 && B.stride(1) == 1,
               "gemm_glu: A [M,K], B [N,K] bf16, K-major");
-  TORCH_CHECK((B.size(0) % 16) == 0 && (act == 0 || act == 1), "gemm_glu: N a multiple of 16, act 0 (silu) or 1 (tanh-gelu)");
-  if (g_decode_gemm && static_b && ferrl::decode_gemm_supported(A.size(0), B.size(0), A.size(1), true))
+  TORCH_CHECK((B.size(0) % 16) == 0 && act >= 0 && act <= 2, "gemm_glu: N a multiple of 16, act 0 (silu), 1 (tanh-gelu) or 2 (clipped)");
+  if (g_decode_gemm && static_b && act < 2 && ferrl::decode_gemm_supported(A.size(0), B.size(0), A.size(1), true))
     return decode_gemm(A, B, optional<Tensor>(), act, 0, true);
   c10::cuda::CUDAGuard guard(A.device());
   ferrl::GemmArgs a{};
@@ -298,6 +298,7 @@ Tensor gemm_glu(const Tensor& A, const Tensor& B, int64_t act, bool static_b) {
   a.out = out.data_ptr(); a.ldo = out.stride(0);
   a.status = status_word(); a.num_sms = num_sms();
   a.glu_act = static_cast<int>(act) + 1;
+  a.glu_alpha = alpha; a.glu_limit = limit;
   a.pdl = (static_b && a.M <= 256) ? 1 : 0;
   int bn = 0, split = 1, cluster = 1;
   ferrl::gemm_plan(a.M, a.N, a.K, 0, a.num_sms, &bn, &split, &cluster, nullptr);
@@ -644,7 +645,7 @@ std::tuple<Tensor, Tensor> gdn_chunk_fwd(const Tensor& q, const Tensor& k, const
   return {out, S};
 }
 
-Tensor glu_fwd(const Tensor& gu, int64_t act);
+Tensor glu_fwd(const Tensor& gu, int64_t act, double alpha = 0.0, double limit = 0.0);
 
 // ---------------------------------------------------------------- mixture of experts
 // logits [T, E] fp32 -> (probs [T,E] f32, scores [T,k] f32, idx [T,k] i32, counts [E] i32)
@@ -977,23 +978,28 @@ void kv_append_paged(const Tensor& k, const Tensor& v, Tensor kc, Tensor vc, con
                                      kc.size(2) * kc.size(3), stream()));
 }
 
-Tensor glu_fwd(const Tensor& gu, int64_t act) {
+static ferrl::GluAct glu_act(int64_t act, double alpha, double limit) {
+  TORCH_CHECK(act >= ferrl::kActSilu && act <= ferrl::kActClipped && (act != ferrl::kActClipped || limit >= 0), "glu: unknown activation");
+  return ferrl::GluAct{static_cast<int>(act), static_cast<float>(alpha), static_cast<float>(limit)};
+}
+
+Tensor glu_fwd(const Tensor& gu, int64_t act, double alpha, double limit) {
   TORCH_CHECK(gu.is_cuda() && gu.is_contiguous(), "glu: contiguous CUDA tensor");
   c10::cuda::CUDAGuard guard(gu.device());
   const int F = gu.size(-1) / 2;
   auto sizes = gu.sizes().vec();
   sizes.back() = F;
   Tensor out = out_empty(sizes, gu.options());
-  FERRL_CHECK(ferrl::glu(dt(gu), false, gu.data_ptr(), nullptr, out.data_ptr(), gu.numel() / (2 * F), F, act, stream()));
+  FERRL_CHECK(ferrl::glu(dt(gu), false, gu.data_ptr(), nullptr, out.data_ptr(), gu.numel() / (2 * F), F, glu_act(act, alpha, limit), stream()));
   return out;
 }
 
-Tensor glu_bwd(const Tensor& gu, const Tensor& dout, int64_t act) {
+Tensor glu_bwd(const Tensor& gu, const Tensor& dout, int64_t act, double alpha, double limit) {
   TORCH_CHECK(gu.is_contiguous() && dout.is_contiguous(), "glu_bwd: contiguous");
   c10::cuda::CUDAGuard guard(gu.device());
   const int F = gu.size(-1) / 2;
   Tensor dgu = out_empty_like(gu);
-  FERRL_CHECK(ferrl::glu(dt(gu), true, gu.data_ptr(), dout.data_ptr(), dgu.data_ptr(), gu.numel() / (2 * F), F, act, stream()));
+  FERRL_CHECK(ferrl::glu(dt(gu), true, gu.data_ptr(), dout.data_ptr(), dgu.data_ptr(), gu.numel() / (2 * F), F, glu_act(act, alpha, limit), stream()));
   return dgu;
 }
 
@@ -1255,6 +1261,209 @@ Tensor latent_decode(const Tensor& q, const Tensor& uk_t, const Tensor& uv, cons
   Tensor out = out_empty({a.B, a.heads * vdim}, q.options());
   FERRL_CHECK(ferrl::head_gemm(a.dtype, ctx.data_ptr(), static_cast<long long>(a.heads) * a.rank, a.rank, uv.data_ptr(), out.data_ptr(),
                                a.heads * vdim, a.B, a.heads, vdim, a.rank, stream()));
+  return out;
+}
+
+// ---------------------------------------------------------------- hyper-connections (csrc/kernels/hyper.cu)
+static bool given(const optional<Tensor>& t) { return t.has_value() && t->defined(); }
+
+// x [rows, ns, W] f32, rewritten in place when y is given and `store` is set; returns h [rows, W]
+Tensor hyper_norm(Tensor x, const optional<Tensor>& y, const optional<Tensor>& mix, const optional<Tensor>& out, const optional<Tensor>& in,
+                  const Tensor& w, double eps, double scale, bool cast_bf16, bool store) {
+  TORCH_CHECK(x.is_cuda() && x.scalar_type() == at::kFloat && x.is_contiguous() && x.dim() == 3 && x.size(1) > 0 && x.size(2) > 0,
+              "hyper_norm: x f32 [rows, streams, W]");
+  c10::cuda::CUDAGuard guard(x.device());
+  ferrl::HyperNormArgs a{};
+  a.rows = x.size(0); a.ns = x.size(1); a.W = x.size(2); a.x = x.data_ptr<float>();
+  a.h_dtype = a.y_dtype = cast_bf16 ? ferrl::kBF16 : ferrl::kF32;
+  if (given(y)) {
+    TORCH_CHECK(y->is_cuda() && y->dim() == 2 && y->size(0) == a.rows && y->size(1) == a.W && y->stride(1) == 1 && dt(*y) == a.y_dtype && given(mix) &&
+                    given(out), "hyper_norm: y [rows, W] in the compute dtype, with its coefficients");
+    f32_vec(*mix, a.ns * a.ns, "hyper_norm: mix f32 [streams, streams]");
+    f32_vec(*out, a.ns, "hyper_norm: out f32 [streams]");
+    a.y = y->data_ptr(); a.ld_y = y->stride(0); a.mix = mix->data_ptr<float>(); a.out = out->data_ptr<float>();
+  }
+  if (given(in)) {
+    f32_vec(*in, a.ns, "hyper_norm: in f32 [streams]");
+    a.in = in->data_ptr<float>();
+  }
+  f32_vec(w, a.W, "hyper_norm: weight f32 [W]");
+  a.w = w.data_ptr<float>(); a.eps = eps; a.scale = scale; a.store = store ? 1 : 0;
+  Tensor h = out_empty({a.rows, a.W}, x.options().dtype(cast_bf16 ? at::kBFloat16 : at::kFloat));
+  a.h = h.data_ptr();
+  FERRL_CHECK(ferrl::hyper_norm(a, stream()));
+  return h;
+}
+
+// ids int64 [n] -> [n, streams, W] f32; token t is at position kv_len[t], or pos[t % pos.numel()]
+Tensor embed_streams(const Tensor& ids, const Tensor& table, const Tensor& pe, const optional<Tensor>& pos, const optional<Tensor>& kv_len, int64_t ns) {
+  TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == at::kLong && ids.dim() == 1 && ids.is_contiguous() && table.dim() == 2 && table.is_contiguous() &&
+                  pe.scalar_type() == at::kFloat && pe.dim() == 2 && pe.is_contiguous() && pe.size(1) == table.size(1) && pe.size(0) > 0 && ns > 0,
+              "embed_streams: ids [n], table [V, W], positions f32 [max_pos, W]");
+  TORCH_CHECK(given(pos) != given(kv_len), "embed_streams: one kind of positions");
+  c10::cuda::CUDAGuard guard(table.device());
+  const long long* pp = nullptr;
+  const int* kp = nullptr;
+  long long S = 1;
+  if (given(pos)) {
+    TORCH_CHECK(pos->is_cuda() && pos->scalar_type() == at::kLong && pos->is_contiguous() && pos->numel() > 0, "embed_streams: positions int64");
+    pp = reinterpret_cast<const long long*>(pos->data_ptr<int64_t>());
+    S = pos->numel();
+  } else {
+    TORCH_CHECK(kv_len->is_cuda() && kv_len->scalar_type() == at::kInt && kv_len->is_contiguous() && kv_len->numel() == ids.numel(), "embed_streams: kv_len int32");
+    kp = kv_len->data_ptr<int>();
+  }
+  Tensor out = out_empty({ids.numel(), ns, table.size(1)}, table.options().dtype(at::kFloat));
+  FERRL_CHECK(ferrl::embed_streams(dt(table), reinterpret_cast<const long long*>(ids.data_ptr<int64_t>()), table.data_ptr(), pe.data_ptr<float>(), pp, kp, S,
+                                   out.data_ptr<float>(), ids.numel(), table.size(1), ns, table.size(0), pe.size(0), stream()));
+  return out;
+}
+
+// ---------------------------------------------------------------- state-space duality layers (csrc/kernels/ssm.cu)
+// batch and token strides of a [B, S, C] operand with packed columns; a size-1 dimension has an arbitrary stride
+static void seq_strides(const Tensor& t, long long* bs, long long* ts) {
+  *ts = t.size(1) > 1 ? t.stride(1) : (t.size(0) > 1 ? t.stride(0) : (t.size(2) + 7) / 8 * 8);
+  *bs = t.size(0) > 1 ? t.stride(0) : *ts * t.size(1);
+}
+
+Tensor ssm_conv(const Tensor& x, const Tensor& w, const optional<Tensor>& bias) {
+  TORCH_CHECK(x.is_cuda() && x.dim() == 3 && x.stride(2) == 1 && w.dim() == 2 && w.size(0) == x.size(2), "ssm_conv: x [B,L,C], w [C,K]");
+  c10::cuda::CUDAGuard guard(x.device());
+  f32_vec(w, w.numel(), "ssm_conv: weight f32 [C, K]");
+  if (given(bias)) f32_vec(*bias, x.size(2), "ssm_conv: bias f32 [C]");
+  long long bs, ts;
+  seq_strides(x, &bs, &ts);
+  Tensor y = out_empty(x.sizes(), x.options());
+  FERRL_CHECK(ferrl::ssm_conv(dt(x), x.data_ptr(), bs, ts, w.data_ptr<float>(), given(bias) ? bias->data_ptr<float>() : nullptr, y.data_ptr(), x.size(0),
+                              x.size(1), x.size(2), w.size(1), stream()));
+  return y;
+}
+
+// u [B, T, H*P + 2*G*N] (x, B and C behind the convolution), dt raw [B, T, H] -> (y [B, T, H*P], state f32 [B, H, N, P])
+std::tuple<Tensor, Tensor> ssm_scan(const Tensor& u, const Tensor& dtr, const Tensor& dt_bias, const Tensor& A_log, const Tensor& D,
+                                    const optional<Tensor>& lens, int64_t heads, int64_t state, int64_t groups, int64_t variant) {
+  TORCH_CHECK(u.is_cuda() && u.dim() == 3 && u.stride(2) == 1 && dtr.dim() == 3 && dtr.stride(2) == 1 && dtr.size(0) == u.size(0) &&
+                  dtr.size(1) == u.size(1) && dtr.size(2) == heads && dtr.scalar_type() == u.scalar_type() && heads > 0 && groups > 0 &&
+                  heads % groups == 0 && state > 0 && (u.size(2) - 2 * groups * state) > 0 && (u.size(2) - 2 * groups * state) % heads == 0,
+              "ssm_scan: u [B,T,H*P+2*G*N], dt [B,T,H]");
+  c10::cuda::CUDAGuard guard(u.device());
+  ferrl::SsmScanArgs a{};
+  a.dtype = dt(u);
+  a.B = u.size(0); a.T = u.size(1); a.H = heads; a.N = state; a.G = groups; a.P = (u.size(2) - 2 * groups * state) / heads;
+  const int64_t es = u.element_size(), inner = heads * a.P;
+  seq_strides(u, &a.bs, &a.ts);
+  seq_strides(dtr, &a.dt_bs, &a.dt_ts);
+  a.x = u.data_ptr();
+  a.Bm = static_cast<const char*>(u.data_ptr()) + inner * es;
+  a.Cm = static_cast<const char*>(u.data_ptr()) + (inner + groups * state) * es;
+  a.dt = dtr.data_ptr();
+  f32_vec(dt_bias, heads, "ssm_scan: dt bias f32 [H]");
+  f32_vec(A_log, heads, "ssm_scan: A_log f32 [H]");
+  f32_vec(D, heads, "ssm_scan: D f32 [H]");
+  a.dt_bias = dt_bias.data_ptr<float>(); a.A_log = A_log.data_ptr<float>(); a.D = D.data_ptr<float>();
+  if (given(lens)) {
+    TORCH_CHECK(lens->is_cuda() && lens->scalar_type() == at::kLong && lens->is_contiguous() && lens->numel() == a.B, "ssm_scan: lens int64 [B]");
+    a.lens = reinterpret_cast<const long long*>(lens->data_ptr<int64_t>());
+  }
+  Tensor y = out_empty({a.B, a.T, inner}, u.options());
+  Tensor S = out_empty({a.B, a.H, a.N, a.P}, u.options().dtype(at::kFloat));
+  a.y = y.data_ptr(); a.state = S.data_ptr<float>();
+  (void)variant;
+  FERRL_CHECK(ferrl::ssm_scan(a, stream()));
+  return {y, S};
+}
+
+Tensor ssm_step(const Tensor& x, const Tensor& dtr, const Tensor& conv_w, const optional<Tensor>& conv_b, const Tensor& dt_bias, const Tensor& A_log,
+                const Tensor& D, Tensor ring, Tensor S, const Tensor& kv_len, const optional<Tensor>& active, int64_t groups) {
+  TORCH_CHECK(S.is_cuda() && S.scalar_type() == at::kFloat && S.dim() == 4 && S.is_contiguous(), "ssm_step: state f32 [B,H,N,P]");
+  c10::cuda::CUDAGuard guard(S.device());
+  ferrl::SsmStepArgs a{};
+  a.dtype = dt(x);
+  a.B = S.size(0); a.H = S.size(1); a.N = S.size(2); a.P = S.size(3); a.G = groups;
+  a.C = a.H * a.P + 2 * a.G * a.N;
+  TORCH_CHECK(groups > 0 && a.H % a.G == 0 && x.dim() == 2 && x.size(0) == a.B && x.size(1) == a.C && x.stride(1) == 1 && dtr.dim() == 2 &&
+                  dtr.size(0) == a.B && dtr.size(1) == a.H && dtr.stride(1) == 1 && dtr.scalar_type() == x.scalar_type(), "ssm_step: x [B,C], dt [B,H]");
+  TORCH_CHECK(conv_w.dim() == 2 && conv_w.size(0) == a.C && conv_w.size(1) > 0, "ssm_step: conv weight [C,K]");
+  a.K = conv_w.size(1);
+  f32_vec(conv_w, conv_w.numel(), "ssm_step: conv weight f32");
+  if (given(conv_b)) f32_vec(*conv_b, a.C, "ssm_step: conv bias f32");
+  f32_vec(dt_bias, a.H, "ssm_step: dt bias f32 [H]");
+  f32_vec(A_log, a.H, "ssm_step: A_log f32 [H]");
+  f32_vec(D, a.H, "ssm_step: D f32 [H]");
+  TORCH_CHECK(ring.is_cuda() && ring.dim() == 3 && ring.is_contiguous() && ring.size(0) == a.B && ring.size(1) == a.K && ring.size(2) == a.C &&
+                  ring.scalar_type() == x.scalar_type(), "ssm_step: ring [B,K,C]");
+  TORCH_CHECK(kv_len.is_cuda() && kv_len.scalar_type() == at::kInt && kv_len.is_contiguous() && kv_len.numel() == a.B, "ssm_step: kv_len int32 [B]");
+  if (given(active)) {
+    TORCH_CHECK(active->is_cuda() && active->scalar_type() == at::kBool && active->is_contiguous() && active->numel() == a.B, "ssm_step: active bool [B]");
+    a.active = reinterpret_cast<const unsigned char*>(active->data_ptr<bool>());
+  }
+  a.x = x.data_ptr(); a.ld_x = x.stride(0); a.dt = dtr.data_ptr(); a.ld_dt = dtr.stride(0);
+  a.conv_w = conv_w.data_ptr<float>(); a.conv_b = given(conv_b) ? conv_b->data_ptr<float>() : nullptr;
+  a.dt_bias = dt_bias.data_ptr<float>(); a.A_log = A_log.data_ptr<float>(); a.D = D.data_ptr<float>();
+  a.ring = ring.data_ptr(); a.state = S.data_ptr<float>(); a.kv_len = kv_len.data_ptr<int>();
+  Tensor y = out_empty({a.B, static_cast<int64_t>(a.H) * a.P}, x.options());
+  a.y = y.data_ptr();
+  FERRL_CHECK(ferrl::ssm_step(a, stream()));
+  return y;
+}
+
+Tensor gated_group_norm(const Tensor& y, const Tensor& z, const Tensor& w, int64_t groups, double eps) {
+  TORCH_CHECK(y.is_cuda() && y.dim() == 2 && y.stride(1) == 1 && z.sizes() == y.sizes() && z.stride(1) == 1 && z.scalar_type() == y.scalar_type(),
+              "gated_group_norm: y, z [rows, W]");
+  c10::cuda::CUDAGuard guard(y.device());
+  f32_vec(w, y.size(1), "gated_group_norm: weight f32 [W]");
+  Tensor out = out_empty(y.sizes(), y.options());
+  FERRL_CHECK(ferrl::gated_group_norm(dt(y), y.data_ptr(), y.stride(0), z.data_ptr(), z.stride(0), w.data_ptr<float>(), out.data_ptr(), y.size(0),
+                                      y.size(1), groups, eps, stream()));
+  return out;
+}
+
+// ---------------------------------------------------------------- distance-biased attention (csrc/kernels/bias_attn.cu)
+// q [B,S,Hq,D], k [B,S,Hkv,D] (also the values), bias f32 [Hq, n]: n distances, at least min(window, S); variant 1 forces the any-size kernel
+Tensor bias_fwd(const Tensor& q, const Tensor& k, const Tensor& bias, double scale, int64_t window, int64_t variant) {
+  TORCH_CHECK(q.is_cuda() && q.dim() == 4 && q.stride(3) == 1 && q.stride(2) == q.size(3) && k.dim() == 4 && k.stride(3) == 1 &&
+                  k.stride(2) == k.size(3) && k.scalar_type() == q.scalar_type() && k.size(0) == q.size(0) && k.size(1) == q.size(1) &&
+                  k.size(3) == q.size(3) && k.size(2) > 0 && q.size(2) % k.size(2) == 0 && window > 0, "bias_fwd: q [B,S,Hq,D], k [B,S,Hkv,D]");
+  TORCH_CHECK(bias.is_cuda() && bias.scalar_type() == at::kFloat && bias.dim() == 2 && bias.is_contiguous() && bias.size(0) == q.size(2) &&
+                  bias.size(1) >= std::min<int64_t>(window, q.size(1)), "bias_fwd: bias f32 [Hq, distances]");
+  c10::cuda::CUDAGuard guard(q.device());
+  ferrl::BiasFwdArgs a{};
+  a.dtype = dt(q);
+  a.B = q.size(0); a.S = q.size(1); a.Hq = q.size(2); a.Hkv = k.size(2); a.D = q.size(3); a.window = std::min<int64_t>(window, q.size(1)); a.scale = scale;
+  a.q = q.data_ptr(); a.k = k.data_ptr(); a.bias = bias.data_ptr<float>(); a.bias_ld = bias.size(1);
+  seq_strides(q.flatten(2), &a.q_bs, &a.q_ts);
+  seq_strides(k.flatten(2), &a.k_bs, &a.k_ts);
+  Tensor out = out_empty({a.B, a.S, static_cast<int64_t>(a.Hq) * a.D}, q.options());
+  a.out = out.data_ptr();
+  (void)variant;
+  FERRL_CHECK(ferrl::bias_fwd_any(a, stream()));
+  return out;
+}
+
+// one token per row: q [B, Hq*D], k [B, Hkv*D] (stored to its ring slot), cache [B, slots, Hkv*D] -> [B, Hq*D]
+Tensor bias_decode(const Tensor& q, const Tensor& k, Tensor cache, const Tensor& kv_len, const optional<Tensor>& active, const Tensor& bias,
+                   int64_t heads, int64_t dim, double scale, int64_t variant) {
+  TORCH_CHECK(q.is_cuda() && q.dim() == 2 && q.stride(1) == 1 && k.dim() == 2 && k.stride(1) == 1 && k.scalar_type() == q.scalar_type() &&
+                  q.size(1) == heads * dim && k.size(1) % dim == 0 && k.size(1) > 0 && heads % (k.size(1) / dim) == 0 && cache.is_cuda() && cache.dim() == 3 &&
+                  cache.is_contiguous() && cache.size(0) == q.size(0) && k.size(0) == q.size(0) && cache.size(1) > 0 && cache.size(2) == k.size(1) &&
+                  cache.scalar_type() == q.scalar_type(), "bias_decode: q [B,Hq*D], k [B,Hkv*D], cache [B,slots,Hkv*D]");
+  TORCH_CHECK(bias.is_cuda() && bias.scalar_type() == at::kFloat && bias.dim() == 2 && bias.is_contiguous() && bias.size(0) == heads &&
+                  bias.size(1) >= cache.size(1), "bias_decode: bias f32 [Hq, slots]");
+  TORCH_CHECK(kv_len.is_cuda() && kv_len.scalar_type() == at::kInt && kv_len.is_contiguous() && kv_len.numel() == q.size(0), "bias_decode: kv_len int32 [B]");
+  c10::cuda::CUDAGuard guard(q.device());
+  ferrl::BiasDecodeArgs a{};
+  a.dtype = dt(q);
+  a.B = q.size(0); a.Hq = heads; a.D = dim; a.Hkv = k.size(1) / dim; a.scale = scale; a.slots = cache.size(1);
+  a.q = q.data_ptr(); a.ld_q = q.stride(0); a.k = k.data_ptr(); a.ld_k = k.stride(0); a.cache = cache.data_ptr();
+  a.kv_len = kv_len.data_ptr<int>(); a.bias = bias.data_ptr<float>(); a.bias_ld = bias.size(1);
+  if (given(active)) {
+    TORCH_CHECK(active->is_cuda() && active->scalar_type() == at::kBool && active->is_contiguous() && active->numel() == a.B, "bias_decode: active bool [B]");
+    a.active = reinterpret_cast<const unsigned char*>(active->data_ptr<bool>());
+  }
+  Tensor out = out_empty({a.B, heads * dim}, q.options());
+  a.out = out.data_ptr();
+  (void)variant;
+  FERRL_CHECK(ferrl::bias_decode_any(a, stream()));
   return out;
 }
 
@@ -1648,8 +1857,8 @@ TORCH_LIBRARY(ferrl_b200, m) {
   m.def("qk_norm_rope_bwd(Tensor q, Tensor k, Tensor? qw, Tensor? kw, Tensor cos, Tensor sin, Tensor pos, int pos_div, float eps, bool zc, Tensor dq, Tensor dk, Tensor(a!) dq_in, Tensor(b!) dk_in) -> ()", &qk_norm_rope_bwd);
   m.def("kv_append(Tensor k, Tensor v, Tensor(a!) kc, Tensor(b!) vc, Tensor kv_len) -> ()", &kv_append);
   m.def("kv_append_paged(Tensor k, Tensor v, Tensor(a!) kc, Tensor(b!) vc, Tensor kv_len, Tensor table) -> ()", &kv_append_paged);
-  m.def("glu_fwd(Tensor gu, int act) -> Tensor", &glu_fwd);
-  m.def("glu_bwd(Tensor gu, Tensor dout, int act) -> Tensor", &glu_bwd);
+  m.def("glu_fwd(Tensor gu, int act, float alpha=0.0, float limit=0.0) -> Tensor", &glu_fwd);
+  m.def("glu_bwd(Tensor gu, Tensor dout, int act, float alpha=0.0, float limit=0.0) -> Tensor", &glu_bwd);
   m.def("embedding(Tensor ids, Tensor table, float scale) -> Tensor", &embedding);
   m.def("lora_merge(Tensor w, Tensor a, Tensor b) -> Tensor", &lora_merge);
   m.def("adamw_step(Tensor[] params, Tensor[] grads, Tensor[] m, Tensor[] v, float lr, float b1, float b2, float eps, float wd, int step, float max_norm, float pre_scale, bool compute_norm) -> Tensor", &adamw_step);
@@ -1660,11 +1869,19 @@ TORCH_LIBRARY(ferrl_b200, m) {
   m.def("latent_append(Tensor(a!) q, Tensor dkv, Tensor norm_w, float eps, Tensor cos_t, Tensor sin_t, Tensor kv_len, Tensor(b!) cache, int dim, int rank) -> ()", &latent_append);
   m.def("latent_fwd(Tensor q, Tensor kv, Tensor lat, int dim, int vdim, int rank, float scale, int window, Tensor? sink, int variant=0) -> Tensor", &latent_fwd);
   m.def("latent_decode(Tensor q, Tensor uk_t, Tensor uv, Tensor cache, Tensor count, float scale, Tensor? sink, int splits=0) -> Tensor", &latent_decode);
+  m.def("hyper_norm(Tensor(a!) x, Tensor? y, Tensor? mix, Tensor? out, Tensor? inp, Tensor w, float eps, float scale, bool cast_bf16, bool store) -> Tensor", &hyper_norm);
+  m.def("embed_streams(Tensor ids, Tensor table, Tensor pe, Tensor? pos, Tensor? kv_len, int streams) -> Tensor", &embed_streams);
+  m.def("ssm_conv(Tensor x, Tensor w, Tensor? bias) -> Tensor", &ssm_conv);
+  m.def("ssm_scan(Tensor u, Tensor dt, Tensor dt_bias, Tensor A_log, Tensor D, Tensor? lens, int heads, int state, int groups, int variant=0) -> (Tensor, Tensor)", &ssm_scan);
+  m.def("ssm_step(Tensor x, Tensor dt, Tensor conv_w, Tensor? conv_b, Tensor dt_bias, Tensor A_log, Tensor D, Tensor(a!) ring, Tensor(b!) S, Tensor kv_len, Tensor? active, int groups) -> Tensor", &ssm_step);
+  m.def("gated_group_norm(Tensor y, Tensor z, Tensor w, int groups, float eps) -> Tensor", &gated_group_norm);
+  m.def("bias_fwd(Tensor q, Tensor k, Tensor bias, float scale, int window, int variant=0) -> Tensor", &bias_fwd);
+  m.def("bias_decode(Tensor q, Tensor k, Tensor(a!) cache, Tensor kv_len, Tensor? active, Tensor bias, int heads, int dim, float scale, int variant=0) -> Tensor", &bias_decode);
   m.def("post_norm(Tensor x, Tensor? y, Tensor? gate, Tensor? gate_bias, Tensor w, Tensor? b, float eps, float alpha, Tensor? history, Tensor? coef, bool cast_bf16, Tensor? r_out) -> (Tensor, Tensor, Tensor)", &post_norm);
   m.def("moe_experts_any(Tensor x, Tensor w, Tensor idx, Tensor counts, Tensor gate_up, Tensor down, int act, bool weight_input) -> Tensor", &moe_experts_any);
   m.def("gemm_norm(Tensor A, Tensor B, Tensor? residual, Tensor? ss_in, float eps, int glu_act, bool want_ss, bool static_b=True) -> (Tensor, Tensor)", &gemm_norm);
   m.def("row_sumsq(Tensor x) -> Tensor", &row_sumsq);
-  m.def("gemm_glu(Tensor A, Tensor B, int act, bool static_b=False) -> Tensor", &gemm_glu);
+  m.def("gemm_glu(Tensor A, Tensor B, int act, bool static_b=False, float alpha=0.0, float limit=0.0) -> Tensor", &gemm_glu);
   m.def("qk_norm_rope_append(Tensor q, Tensor k, Tensor v, Tensor? qw, Tensor? kw, Tensor cos_t, Tensor sin_t, Tensor pos, float eps, bool zc, Tensor(a!) kc, Tensor(b!) vc, Tensor kv_len, Tensor? table) -> Tensor", &qk_norm_rope_append);
   m.def("flash_fwd(Tensor q, Tensor k, Tensor v, float scale, bool causal, int window, int q_offset, int variant=0) -> (Tensor, Tensor)", &flash_fwd);
   m.def("flash_bwd(Tensor q, Tensor k, Tensor v, Tensor o, Tensor lse, Tensor d_o, float scale, bool causal, int window, int q_offset, int variant=0, Tensor? debug=None) -> (Tensor, Tensor, Tensor)", &flash_bwd);

@@ -93,7 +93,7 @@ struct GemmParams {
   // Gated-linear-unit epilogue (one-SM kernel, bf16 output, no k-split): the N rows of B come in groups
   // of 16, eight gate rows followed by the eight up rows of the same features, and the kernel writes
   // act(gate) * up, N / 2 columns per row.  1 = SiLU, 2 = tanh-GELU.
-  int glu_act;
+  int glu_act; float glu_alpha, glu_limit;
   // Language-model head without a logits tensor (one-SM kernel with 256-wide tiles and the two-SM kernel).
   // Every accumulator value is first turned into the scored logit z = softcap(x) / T.
   //   lp_mode 1: nothing is stored to `out`; per row and column tile the epilogue writes the running
@@ -760,6 +760,11 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUt
                 for (int e = 0; e < 8; ++e) {
                   const float gate = __uint_as_float(r[g16 * 16 + e]), up = __uint_as_float(r[g16 * 16 + 8 + e]);
                   float a;
+                  if (p.glu_act == 3) {
+                    const float gc = fminf(gate, p.glu_limit), uc = fminf(fmaxf(up, -p.glu_limit), p.glu_limit);
+                    o8[e] = gc / (1.f + __expf(-p.glu_alpha * gc)) * (uc + 1.f);
+                    continue;
+                  }
                   if (p.glu_act == 1) {
                     a = gate / (1.f + __expf(-gate));
                   } else {
@@ -1183,6 +1188,8 @@ const char* launch_bn(const GemmArgs& a, cudaStream_t stream) {
   p.partial = a.partial;
   p.tile_expert = a.tile_expert;
   p.glu_act = a.glu_act;
+  p.glu_alpha = a.glu_alpha;
+  p.glu_limit = a.glu_limit;
   p.ss_in = a.ss_in; p.ss_parts = a.ss_parts; p.ss_ld = a.ss_ld; p.ss_inv_k = a.ss_inv_k; p.ss_eps = a.ss_eps;
   p.ss_out = a.ss_out;
   p.lp_mode = a.lp_mode; p.lp_targets = a.lp_targets; p.lp_inv_t = a.lp_inv_t; p.lp_cap = a.lp_cap; p.lp_col0 = a.lp_col0;

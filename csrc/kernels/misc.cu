@@ -29,9 +29,27 @@ __device__ __forceinline__ float act_grad(float g, int act) {
   return 0.5f * (1.f + t) + 0.5f * g * (1.f - t * t) * du;
 }
 
+// act(g) * u and its derivatives by g and u
+__device__ __forceinline__ float glu_f(float g, float u, const GluAct& k) {
+  if (k.act == kActClipped) {
+    g = fminf(g, k.limit);
+    u = fminf(fmaxf(u, -k.limit), k.limit);
+    return g / (1.f + __expf(-k.alpha * g)) * (u + 1.f);
+  }
+  return act_fwd(g, k.act) * u;
+}
+__device__ __forceinline__ float2 glu_grad(float g, float u, const GluAct& k) {
+  if (k.act == kActClipped) {
+    const float gc = fminf(g, k.limit), uc = fminf(fmaxf(u, -k.limit), k.limit);
+    const float s = 1.f / (1.f + __expf(-k.alpha * gc));
+    return make_float2(g > k.limit ? 0.f : s * (1.f + k.alpha * gc * (1.f - s)) * (uc + 1.f), fabsf(u) > k.limit ? 0.f : gc * s);
+  }
+  return make_float2(u * act_grad(g, k.act), act_fwd(g, k.act));
+}
+
 // gate_up [rows, 2F] laid out [gate | up] -> out [rows, F]
 template <typename T>
-__global__ void glu_fwd_kernel(const T* __restrict__ gu, T* __restrict__ out, long long rows, int F, int act) {
+__global__ void glu_fwd_kernel(const T* __restrict__ gu, T* __restrict__ out, long long rows, int F, GluAct act) {
   pdl_trigger();   // a dependent GEMM may start streaming its weights while this kernel runs
   pdl_wait();      // launched as a programmatic dependent itself: nothing is read before the predecessor is done
   long long n = rows * F;
@@ -41,12 +59,12 @@ __global__ void glu_fwd_kernel(const T* __restrict__ gu, T* __restrict__ out, lo
     int c = static_cast<int>(i - r * F);
     float g = to_f(gu[r * 2 * F + c]);
     float u = to_f(gu[r * 2 * F + F + c]);
-    out[i] = from_f<T>(act_fwd(g, act) * u);
+    out[i] = from_f<T>(glu_f(g, u, act));
   }
 }
 // bf16 vector forms: 8 elements per thread per step, 16-byte loads and stores; F % 8 == 0
 __global__ void glu_fwd_vec_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ out, long long rows,
-                                   int F, int act) {
+                                   int F, GluAct act) {
   pdl_trigger();   // a dependent GEMM may start streaming its weights while this kernel runs
   pdl_wait();      // launched as a programmatic dependent itself: nothing is read before the predecessor is done
   const int chunks = F / 8;
@@ -64,13 +82,13 @@ __global__ void glu_fwd_vec_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bf
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const float2 g = __bfloat1622float2(gh[e]), u = __bfloat1622float2(uh[e]);
-      oh[e] = __floats2bfloat162_rn(act_fwd(g.x, act) * u.x, act_fwd(g.y, act) * u.y);
+      oh[e] = __floats2bfloat162_rn(glu_f(g.x, u.x, act), glu_f(g.y, u.y, act));
     }
     *reinterpret_cast<uint4*>(out + r * F + c * 8) = o;
   }
 }
 __global__ void glu_bwd_vec_kernel(const __nv_bfloat16* __restrict__ gu, const __nv_bfloat16* __restrict__ dout,
-                                   __nv_bfloat16* __restrict__ dgu, long long rows, int F, int act) {
+                                   __nv_bfloat16* __restrict__ dgu, long long rows, int F, GluAct act) {
   const int chunks = F / 8;
   const long long n = rows * chunks;
   for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < n;
@@ -89,8 +107,9 @@ __global__ void glu_bwd_vec_kernel(const __nv_bfloat16* __restrict__ gu, const _
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const float2 g = __bfloat1622float2(gh[e]), u = __bfloat1622float2(uh[e]), d = __bfloat1622float2(dh[e]);
-      ogh[e] = __floats2bfloat162_rn(d.x * u.x * act_grad(g.x, act), d.y * u.y * act_grad(g.y, act));
-      ouh[e] = __floats2bfloat162_rn(d.x * act_fwd(g.x, act), d.y * act_fwd(g.y, act));
+      const float2 dx = glu_grad(g.x, u.x, act), dy = glu_grad(g.y, u.y, act);
+      ogh[e] = __floats2bfloat162_rn(d.x * dx.x, d.y * dy.x);
+      ouh[e] = __floats2bfloat162_rn(d.x * dx.y, d.y * dy.y);
     }
     *reinterpret_cast<uint4*>(dgu + r * 2 * F + c * 8) = og;
     *reinterpret_cast<uint4*>(dgu + r * 2 * F + F + c * 8) = ou;
@@ -99,7 +118,7 @@ __global__ void glu_bwd_vec_kernel(const __nv_bfloat16* __restrict__ gu, const _
 
 template <typename T>
 __global__ void glu_bwd_kernel(const T* __restrict__ gu, const T* __restrict__ dout, T* __restrict__ dgu,
-                               long long rows, int F, int act) {
+                               long long rows, int F, GluAct act) {
   long long n = rows * F;
   for (long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x; i < n;
        i += static_cast<long long>(gridDim.x) * blockDim.x) {
@@ -108,8 +127,9 @@ __global__ void glu_bwd_kernel(const T* __restrict__ gu, const T* __restrict__ d
     float g = to_f(gu[r * 2 * F + c]);
     float u = to_f(gu[r * 2 * F + F + c]);
     float d = to_f(dout[i]);
-    dgu[r * 2 * F + c] = from_f<T>(d * u * act_grad(g, act));
-    dgu[r * 2 * F + F + c] = from_f<T>(d * act_fwd(g, act));
+    const float2 dd = glu_grad(g, u, act);
+    dgu[r * 2 * F + c] = from_f<T>(d * dd.x);
+    dgu[r * 2 * F + F + c] = from_f<T>(d * dd.y);
   }
 }
 
@@ -285,7 +305,7 @@ inline unsigned grid_for(long long n, int threads) {
 
 }  // namespace
 
-const char* glu(int dtype, bool backward, const void* gu, const void* dout, void* out, long long rows, int F, int act,
+const char* glu(int dtype, bool backward, const void* gu, const void* dout, void* out, long long rows, int F, GluAct act,
                 cudaStream_t s) {
   if (rows * F == 0) return nullptr;
   unsigned grid = grid_for(rows * F, 256);

@@ -304,9 +304,13 @@ class GraphedDecodeStep:
             # one eager step warms every kernel (and lazy one-time allocations) before capture; its
             # effects are rolled back so the captured graph starts from the same state
             snap = (self.logits.clone(),)
+            state = [(t, t.clone()) for t in (self.dec.step_state() if hasattr(self.dec, "step_state") else ())]
             self._body()
             torch.cuda.synchronize()
             self.dec.kv_len.copy_(kv0)
+            for t, kept in state:           # recurrent layers: repeating the step would advance them twice
+                t.copy_(kept)
+            del state
             self.logits.copy_(snap[0])
             self.draw.zero_()
             self.finished.zero_()

@@ -37,7 +37,7 @@ class LoaderOpts:
     full_ft: bool = False
     adapter_seed: int = 0
     max_position_embeddings: Optional[int] = None
-    gdn_targets: str = ""     # hybrid families: adapted GatedDeltaNet projections, letters of q z b a o (see qwen35.py)
+    gdn_targets: str = ""     # hybrid families: adapted recurrent-layer projections, letters of q z b a o (see qwen35.py, mamba2.py)
 
 
 @dataclass(frozen=True)
@@ -243,7 +243,8 @@ def load_auto_policy(model_dir: str, opts: Optional[LoaderOpts] = None):
     ``(model, PolicyLoadIdentity)``.  ``model_type`` dispatch: ``qwen3`` ->
     dense Qwen3, ``qwen3_5``/``qwen3_5_text``/``qwen3_5_moe`` -> hybrid,
     ``gemma4``/``gemma4_text`` -> Gemma; ``architecture`` ``Galodra`` ->
-    latent attention with gated residuals.  Llama must be loaded explicitly with
+    latent attention with gated residuals, ``Mifutar`` -> Mamba-2 and biased
+    attention with hyper-connections.  Llama must be loaded explicitly with
     ``load_llama`` (library API only)."""
     opts = opts or LoaderOpts()
     cfg = read_config(model_dir)
@@ -260,7 +261,10 @@ def load_auto_policy(model_dir: str, opts: Optional[LoaderOpts] = None):
     if mt == "Galodra":
         from .galodra import load_galodra
         return load_galodra(model_dir, opts)
-    raise ValueError(f"unsupported model_type {mt!r} (supported: qwen3, qwen3_5[_moe], gemma4, Galodra)")
+    if mt == "Mifutar":
+        from .mifutar import load_mifutar
+        return load_mifutar(model_dir, opts)
+    raise ValueError(f"unsupported model_type {mt!r} (supported: qwen3, qwen3_5[_moe], gemma4, Galodra, Mifutar)")
 
 
 def load_llama(model_dir: str, opts: Optional[LoaderOpts] = None):

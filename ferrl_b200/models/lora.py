@@ -172,7 +172,7 @@ class FusedLoraLinear(nn.Module):
                  adapted: Sequence[bool], lora: Optional[LoraSpec], *, dtype=torch.float32,
                  device=None, shard: Optional[Shard] = None, full_in: Optional[int] = None,
                  full_out_sizes: Optional[Sequence[int]] = None, keep_transpose: bool = False,
-                 quant: BaseQuantization = BaseQuantization.NONE, trainable_base: bool = False):
+                 quant: BaseQuantization = BaseQuantization.NONE, trainable_base: bool = False, bias: bool = False):
         super().__init__()
         self.in_features = in_features
         self.out_sizes = list(out_sizes)
@@ -189,6 +189,11 @@ class FusedLoraLinear(nn.Module):
             self.weight = nn.Parameter(w)
         else:
             self.register_buffer("weight", w, persistent=False)
+        b = torch.zeros(sum(out_sizes), dtype=dtype, device=device) if bias else None      # single-rank projections only
+        if bias and trainable_base:
+            self.bias = nn.Parameter(b)
+        else:
+            self.register_buffer("bias", b, persistent=False)
         self.register_buffer("weight_t", None, persistent=False)
         self.register_buffer("weight_merged", None, persistent=False)
         self.weight_decode = None               # see enable_decode_fold()
@@ -279,7 +284,7 @@ class FusedLoraLinear(nn.Module):
     # --------------------------------------------------------------- forward
     def forward(self, x: torch.Tensor, residual=None) -> torch.Tensor:
         a, b = self._stacks()
-        return ops.lora_linear(x, self.weight, a, b, wt=self.weight_t, residual=residual)
+        return ops.lora_linear(x, self.weight, a, b, wt=self.weight_t, bias=self.bias, residual=residual)
 
     def forward_reduce(self, x: torch.Tensor, comm, merged: bool = False, residual=None) -> torch.Tensor:
         """Row-parallel use: the projection, its tensor-parallel sum over ``comm`` and an
@@ -351,7 +356,7 @@ class FusedLoraLinear(nn.Module):
     def forward_merged(self, x: torch.Tensor, residual=None) -> torch.Tensor:
         """Rollout path over the merged snapshot (no adapter side path)."""
         w = self.weight_merged if self.weight_merged is not None else self.weight
-        y = ops.lora_linear(x, w, None, None, residual=None if self._glu_rows() is not None else residual)
+        y = ops.lora_linear(x, w, None, None, bias=self.bias, residual=None if self._glu_rows() is not None else residual)
         if self._glu_rows() is not None:      # snapshot rows are interleaved for the fused GLU: undo it for plain use
             y = y.index_select(-1, self._glu_inverse)
             if residual is not None:
@@ -422,11 +427,11 @@ class FusedLoraLinear(nn.Module):
         else:
             self.weight_decode = wd
 
-    def forward_merged_glu(self, x: torch.Tensor, act: str) -> torch.Tensor:
+    def forward_merged_glu(self, x: torch.Tensor, act) -> torch.Tensor:
         """``act(x Wg^T) * (x Wu^T)`` over the merged snapshot; one kernel where the snapshot is
         interleaved, projection + GLU kernel otherwise."""
-        if self._glu_rows() is not None and ops.native(x) and x.dtype == torch.bfloat16 and act in ("silu", "gelu_pytorch_tanh",
-                                                                                                    "gelu_tanh"):
+        if self._glu_rows() is not None and ops.native(x) and x.dtype == torch.bfloat16 and \
+                (isinstance(act, ops.ClippedGlu) or act in ("silu", "gelu_pytorch_tanh", "gelu_tanh")):
             from ..ops import cuda as _c
             return _c.gemm_glu(x, self.weight_merged, act)
         return ops.swiglu(self.forward_merged(x), act)

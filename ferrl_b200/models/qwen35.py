@@ -533,6 +533,10 @@ class Qwen35CachedDecoder:
     def cache_bytes(self) -> int:
         return sum(t.numel() * t.element_size() for s in self.state for t in s)
 
+    def step_state(self):
+        """Tensors that a decode step advances; a step that is taken twice has to start from a copy of them."""
+        return [t for l, st in zip(self.m.layers, self.state) if l.kind == "linear_attention" for t in st]
+
     @torch.no_grad()
     def prefill(self, ids, lens, rows=None, at=None):
         m = self.m

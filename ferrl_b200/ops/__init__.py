@@ -11,8 +11,8 @@ from __future__ import annotations
 import torch
 
 from . import eager
-from .eager import (apply_rope, default_inv_freq, l2norm, llama3_inv_freq, rope_tables,
-                    stable_softplus)
+from .eager import (ClippedGlu, apply_rope, default_inv_freq, hyper_mix, l2norm, llama3_inv_freq, rope_tables,
+                    sinusoid_table, stable_softplus)
 
 
 class ExtensionMissing(RuntimeError):
@@ -147,6 +147,60 @@ def latent_decode(q, uk_t, uv, cache, count, *, rank, scale, sink=None):
     if _on_gpu(q):
         return _cuda().latent_decode(q, uk_t, uv, cache, count, rank=rank, scale=scale, sink=sink)
     return eager.latent_decode(q, uk_t, uv, cache, count, rank=rank, scale=scale, sink=sink)
+
+
+def bias_attention(q, k, bias, *, scale, window):
+    if _on_gpu(q):
+        return _cuda().bias_attention(q, k, bias, scale=scale, window=window)
+    return eager.bias_attention(q, k, bias, scale=scale, window=window)
+
+
+def bias_decode(q, k, cache, kv_len, bias, *, dim, scale, active=None):
+    if _on_gpu(q):
+        return _cuda().bias_decode(q, k, cache, kv_len, bias, dim=dim, scale=scale, active=active)
+    return eager.bias_decode(q, k, cache, kv_len, bias, dim=dim, scale=scale, active=active)
+
+
+def embed_streams(ids, table, pe, positions, streams):
+    """Embedding rows plus position rows, float32, repeated ``streams`` times: ``ids`` ``[B,S]`` with positions ``[S]``, or
+    ``ids`` ``[B]`` with one position per row (``kv_len``, int32).  Returns ``[..., streams, W]``."""
+    if _on_gpu(table):
+        return _cuda().embed_streams(ids, table, pe, positions, streams)
+    x = eager.embedding(ids, table).float() + pe[positions.long()]
+    return x.unsqueeze(-2).expand(*x.shape[:-1], streams, x.shape[-1]).contiguous()
+
+
+def hyper_norm(x, y, mix, out, inp, weight, eps, cast, scale=1.0, store=True):
+    """``eager.hyper_norm`` with ``h`` in the dtype ``cast``.  The kernel rewrites the streams in place (``store=False``:
+    not at all, the returned streams are then stale)."""
+    if _on_gpu(x):
+        return _cuda().hyper_norm(x, y, mix, out, inp, weight, eps, cast, scale, store)
+    x, h = eager.hyper_norm(x, y, mix, out, inp, weight, eps, scale)
+    return x, h.to(cast)
+
+
+def ssm_conv(x, w, bias):
+    if _on_gpu(x):
+        return _cuda().ssm_conv(x, w, bias)
+    return eager.ssm_conv(x, w, bias)
+
+
+def ssm_scan(u, dt, dt_bias, A_log, D, lens, *, heads, state, groups):
+    if _on_gpu(u):
+        return _cuda().ssm_scan(u, dt, dt_bias, A_log, D, lens, heads=heads, state=state, groups=groups)
+    return eager.ssm_scan(u, dt, dt_bias, A_log, D, lens, heads=heads, state=state, groups=groups)
+
+
+def ssm_step(x, dt, conv_w, conv_b, dt_bias, A_log, D, ring, S, kv_len, active, *, groups):
+    if _on_gpu(x):
+        return _cuda().ssm_step(x, dt, conv_w, conv_b, dt_bias, A_log, D, ring, S, kv_len, active, groups=groups)
+    return eager.ssm_step(x, dt, conv_w, conv_b, dt_bias, A_log, D, ring, S, kv_len, active, groups=groups)
+
+
+def gated_group_norm(y, z, weight, groups, eps):
+    if _on_gpu(y):
+        return _cuda().gated_group_norm(y, z, weight, groups, eps)
+    return eager.gated_group_norm(y, z, weight, groups, eps)
 
 
 def linear_f32(x, w):

@@ -67,7 +67,8 @@ def gemm_glu(x, w_interleaved, act="silu"):
     x2 = x.reshape(-1, x.shape[-1])
     if not x2.is_contiguous():
         x2 = x2.contiguous()
-    y = lib().gemm_glu(x2, w_interleaved, _ACT[act], True)
+    a, *par = _glu_act(act)
+    y = lib().gemm_glu(x2, w_interleaved, a, True, *par)
     return y.view(*x.shape[:-1], w_interleaved.shape[0] // 2)
 
 
@@ -300,7 +301,10 @@ def lora_linear_reduce(x, w, a_stack, b_stack, wt, reducer, residual=None):
 
 def lora_linear(x, w, a_stack, b_stack, wt=None, bias=None, residual=None):
     """``x Wᵀ + (x Aᵀ) Bᵀ (+ residual)``; the residual add happens in the GEMM epilogue."""
-    if not (_bf16(x) and _bf16(w)) or bias is not None or w.requires_grad or x.shape[-1] % 8:
+    fits = _bf16(x) and _bf16(w) and not w.requires_grad and x.shape[-1] % 8 == 0
+    if fits and bias is not None and residual is None and _bf16(bias) and not bias.requires_grad:
+        residual, bias = bias.expand(*x.shape[:-1], w.shape[0]), None      # one row that every row adds in the epilogue
+    if not fits or bias is not None:
         y = eager.lora_linear(x, w, a_stack, b_stack, bias)
         return y if residual is None else residual + y
     if residual is not None and residual.dtype != torch.bfloat16:
@@ -626,6 +630,76 @@ def latent_decode(q, uk_t, uv, cache, count, *, rank, scale, sink=None, splits=0
     return lib().latent_decode(q, uk_t, uv if uv.is_contiguous() else uv.contiguous(), cache, count, float(scale), sink, int(splits))
 
 
+# ------------------------------------------------------- distance-biased attention, hyper-connections, state-space duality
+def bias_attention(q, k, bias, *, scale, window, variant=0):
+    """Whole sequences; ``variant=1`` forces the any-size kernel (``csrc/kernels/bias_attn.cu``)."""
+    def native_fn(q_, k_, b_):
+        return lib().bias_fwd(_packed(q_), _packed(k_), b_.contiguous(), float(scale), int(window), int(variant))
+    if _wants_grad(q, k, bias):
+        return _EagerGrad.apply(native_fn, lambda q_, k_, b_: eager.bias_attention(q_, k_, b_, scale=scale, window=window), q, k, bias)
+    return native_fn(q, k, bias)
+
+
+def bias_decode(q, k, cache, kv_len, bias, *, dim, scale, active=None, variant=0):
+    return lib().bias_decode(q, k, cache, kv_len, active, bias, q.shape[-1] // dim, dim, float(scale), int(variant))
+
+
+def embed_streams(ids, table, pe, positions, streams):
+    if table.requires_grad:
+        x = eager.embedding(ids, table).float() + pe[positions.long()]
+        return x.unsqueeze(-2).expand(*x.shape[:-1], streams, x.shape[-1])
+    per_row = positions.dtype == torch.int32
+    out = lib().embed_streams(ids.reshape(-1).contiguous(), table, pe, None if per_row else positions.contiguous(),
+                              positions if per_row else None, streams)
+    return out.view(*ids.shape, streams, table.shape[1])
+
+
+def hyper_norm(x, y, mix, out, inp, weight, eps, cast, scale, store):
+    """See ``csrc/kernels/hyper.cu``; with gradients the eager form, which leaves its input alone."""
+    if _wants_grad(x, y, mix, out, inp, weight):
+        x, h = eager.hyper_norm(x, y, mix, out, inp, weight, eps, scale)
+        return x, h.to(cast)
+    ns, W = x.shape[-2:]
+    h = lib().hyper_norm(x.view(-1, ns, W), None if y is None else _rows2(y, W), mix, out, inp, weight, float(eps), float(scale),
+                         cast == torch.bfloat16, bool(store))
+    return x, h.view(*x.shape[:-2], W)
+
+
+def _cols(t):
+    return t if t.stride(-1) == 1 else t.contiguous()
+
+
+def ssm_conv(x, w, bias):
+    if _wants_grad(x, w, bias):
+        return _EagerGrad.apply(lambda *a: lib().ssm_conv(_cols(a[0]), *a[1:]), eager.ssm_conv, x, w, bias)
+    return lib().ssm_conv(_cols(x), w, bias)
+
+
+def ssm_scan(u, dt, dt_bias, A_log, D, lens, *, heads, state, groups, variant=0):
+    """``variant=1`` forces the float32 kernel of any size."""
+    def native_fn(u_, dt_, b_, a_, d_):
+        return lib().ssm_scan(_cols(u_), _cols(dt_), b_, a_, d_, lens, heads, state, groups, int(variant))
+    if _wants_grad(u, dt, dt_bias, A_log, D):
+        y = _EagerGrad.apply(lambda *a: native_fn(*a)[0], lambda *a: eager.ssm_scan(*a, lens, heads=heads, state=state, groups=groups)[0],
+                             u, dt, dt_bias, A_log, D)
+        return y, None
+    return native_fn(u, dt, dt_bias, A_log, D)
+
+
+def ssm_step(x, dt, conv_w, conv_b, dt_bias, A_log, D, ring, S, kv_len, active, *, groups):
+    return lib().ssm_step(x, dt, conv_w, conv_b, dt_bias, A_log, D, ring, S, kv_len, active, groups)
+
+
+def gated_group_norm(y, z, weight, groups, eps):
+    W = y.shape[-1]
+
+    def native_fn(y_, z_, w_):
+        return lib().gated_group_norm(_rows2(y_, W), _rows2(z_, W), w_, groups, float(eps)).view(y.shape)
+    if _wants_grad(y, z, weight):
+        return _EagerGrad.apply(native_fn, lambda y_, z_, w_: eager.gated_group_norm(y_, z_, w_, groups, eps), y, z, weight)
+    return native_fn(y, z, weight)
+
+
 def linear_f32(x, w):
     """float32 result of a projection: tcgen05 GEMM with an fp32 epilogue for bf16 operands."""
     if _wants_grad(x, w) or not (_bf16(x) and _bf16(w)) or x.shape[-1] % 8:
@@ -640,24 +714,29 @@ def linear_f32(x, w):
 _ACT = {"silu": 0, "gelu_pytorch_tanh": 1, "gelu_tanh": 1}
 
 
+def _glu_act(act):
+    """``(id, alpha, limit)`` of a gated activation."""
+    return (2, float(act.alpha), float(act.limit)) if isinstance(act, eager.ClippedGlu) else (_ACT[act], 0.0, 0.0)
+
+
 class _Glu(torch.autograd.Function):
     @staticmethod
     def forward(ctx, gu, act):
         guc = gu.contiguous()
         ctx.save_for_backward(guc)
         ctx.act = act
-        return lib().glu_fwd(guc, act)
+        return lib().glu_fwd(guc, *act)
 
     @staticmethod
     def backward(ctx, dout):
         (gu,) = ctx.saved_tensors
-        return lib().glu_bwd(gu, dout.contiguous(), ctx.act), None
+        return lib().glu_bwd(gu, dout.contiguous(), *ctx.act), None
 
 
 def swiglu(gate_up, act="silu"):
-    if act not in _ACT:
+    if act not in _ACT and not isinstance(act, eager.ClippedGlu):
         return eager.swiglu(gate_up, act)
-    return _Glu.apply(gate_up, _ACT[act])
+    return _Glu.apply(gate_up, _glu_act(act))
 
 
 # ------------------------------------------------------------------ GatedDeltaNet

@@ -7,6 +7,7 @@ accumulates in float32 and is written the obvious way on purpose.
 from __future__ import annotations
 
 import math
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -253,10 +254,153 @@ def latent_decode(q, uk_t, uv, cache, count, *, rank: int, scale: float, sink=No
     return torch.einsum("bhk,hvk->bhv", ctx, uv.float()).reshape(B, -1).to(q.dtype)
 
 
+# --------------------------------------------- distance-biased attention ----
+def bias_attention(q, k, bias, *, scale: float, window: int):
+    """Causal sliding-window attention whose values are the keys: ``q`` ``[B,S,H,D]``, ``k`` ``[B,S,G,D]``, ``bias``
+    ``[H,n]`` added to the scaled score of every distance ``0 .. min(window, S) - 1``.  Returns ``[B,S,H*D]``."""
+    B, S, H, D = q.shape
+    kf = k.float().repeat_interleave(H // k.shape[2], dim=2)
+    n = torch.arange(S, device=q.device)
+    d = n[:, None] - n[None, :]
+    ok = (d >= 0) & (d < window)
+    scores = torch.einsum("bihd,bjhd->bhij", q.float(), kf) * scale + bias.float()[:, d.clamp(0, bias.shape[1] - 1)]
+    p = torch.softmax(scores.masked_fill(~ok, float("-inf")), dim=-1)
+    return torch.einsum("bhij,bjhd->bihd", p, kf).reshape(B, S, H * D).to(q.dtype)
+
+
+def bias_decode(q, k, cache, kv_len, bias, *, dim: int, scale: float, active=None):
+    """One token per row at position ``kv_len[b]``: ``q`` ``[B,H*dim]``, its own key ``k`` ``[B,G*dim]`` goes to slot
+    ``kv_len[b] % slots`` of the ring ``cache`` ``[B,slots,G*dim]`` (in place).  Rows that are not ``active`` attend to
+    nothing and store nothing.  Returns ``[B,H*dim]``."""
+    B, slots = cache.shape[0], cache.shape[1]
+    pos = kv_len.long()
+    rows = torch.arange(B, device=q.device)
+    cur = pos % slots
+    on = torch.ones(B, dtype=torch.bool, device=q.device) if active is None else active
+    cache[rows, cur] = torch.where(on[:, None], k, cache[rows, cur])
+    qh, kc = q.view(B, -1, dim).float(), cache.view(B, slots, -1, dim).float()
+    kc = kc.repeat_interleave(qh.shape[1] // kc.shape[2], dim=2)
+    dist = (cur[:, None] - torch.arange(slots, device=q.device)[None, :]) % slots
+    ok = (dist <= pos[:, None]) & on[:, None]
+    scores = torch.einsum("bhd,bshd->bhs", qh, kc) * scale + bias.float()[:, dist].transpose(0, 1)
+    p = torch.nan_to_num(torch.softmax(scores.masked_fill(~ok[:, None], float("-inf")), dim=-1))
+    return torch.einsum("bhs,bshd->bhd", p, kc).reshape(B, -1).to(q.dtype)
+
+
+# ---------------------------------------------------- hyper-connections ----
+def sinusoid_table(n: int, width: int) -> torch.Tensor:
+    """``[n, width]`` float32: entry ``2i`` is ``sin(p * 10000^(-2i/width))``, entry ``2i+1`` the cosine."""
+    i = torch.arange((width + 1) // 2, dtype=torch.float64)
+    angle = torch.arange(n, dtype=torch.float64)[:, None] * 10000.0 ** (-2.0 * i / width)
+    return torch.stack([angle.sin(), angle.cos()], dim=-1).reshape(n, -1)[:, :width].float()
+
+
+def hyper_mix(x, y, mix, out):
+    """Streams ``x`` ``[..., s, W]`` behind a sublayer with output ``y`` ``[..., W]``: stream ``t`` becomes
+    ``sum_s mix[s, t] x_s + out[t] y`` (float32)."""
+    return torch.einsum("st,...sw->...tw", mix.float(), x) + out.float()[:, None] * y.float()[..., None, :]
+
+
+def hyper_norm(x, y, mix, out, inp, weight, eps, scale: float = 1.0):
+    """``(streams, h)``: the streams behind the sublayer that gave ``y`` (``None``: as they are), and the RMS norm
+    (weight around zero, times ``scale``) of what the next sublayer reads, ``sum_s inp[s] x_s`` (``inp=None``: the
+    plain sum).  Float32."""
+    if y is not None:
+        x = hyper_mix(x, y, mix, out)
+    u = x.sum(-2) if inp is None else torch.einsum("s,...sw->...w", inp.float(), x)
+    h = u * torch.rsqrt(u.pow(2).mean(-1, keepdim=True) + eps) * (1.0 + weight.float())
+    return x, h if scale == 1.0 else h * scale
+
+
+# ------------------------------------------------ state-space duality ----
+def ssm_conv(x, w, bias):
+    """Causal convolution per channel and SiLU: ``x`` ``[B,L,C]``, ``w`` ``[C,K]`` whose last column meets the current
+    token, zeros before the start."""
+    xf = F.pad(x.float().transpose(1, 2), (w.shape[1] - 1, 0))
+    y = F.conv1d(xf, w.float().unsqueeze(1), None if bias is None else bias.float(), groups=x.shape[2])
+    return F.silu(y).transpose(1, 2).to(x.dtype)
+
+
+def ssm_scan(u, dt, dt_bias, A_log, D, lens, *, heads: int, state: int, groups: int, chunk: int = 64):
+    """Selective scan of ``u = [x | B | C]`` ``[B,T,H*P + 2*G*N]`` with raw step sizes ``dt`` ``[B,T,H]``, in chunks whose
+    products are matrices; float32 inside.  Tokens at or past ``lens[b]`` leave the state alone.  Returns ``(y [B,T,H*P],
+    state [B,H,N,P])``."""
+    Bn, T, _ = u.shape
+    inner = u.shape[2] - 2 * groups * state
+    P, rep = inner // heads, heads // groups
+    uf = u.float()
+    x = uf[..., :inner].reshape(Bn, T, heads, P)
+    Bm = uf[..., inner:inner + groups * state].reshape(Bn, T, groups, state).repeat_interleave(rep, dim=2)
+    Cm = uf[..., inner + groups * state:].reshape(Bn, T, groups, state).repeat_interleave(rep, dim=2)
+    step = F.softplus(dt.float() + dt_bias.float())
+    if lens is not None:
+        step = step * (torch.arange(T, device=u.device)[None, :] < lens[:, None])[..., None]
+    la = -torch.exp(A_log.float()) * step
+    S = x.new_zeros(Bn, heads, state, P)
+    ys = []
+    for t0 in range(0, T, chunk):
+        xc, bc, cc = x[:, t0:t0 + chunk], Bm[:, t0:t0 + chunk], Cm[:, t0:t0 + chunk]
+        cum = la[:, t0:t0 + chunk].cumsum(1).transpose(1, 2)                     # [B,H,L]
+        xs = (xc * step[:, t0:t0 + chunk, :, None]).transpose(1, 2)              # [B,H,L,P]
+        L = cum.shape[-1]
+        seg = cum[..., :, None] - cum[..., None, :]
+        seg = seg.masked_fill(~torch.ones(L, L, dtype=torch.bool, device=u.device).tril(), float("-inf"))
+        scores = torch.einsum("bthn,bshn->bhts", cc, bc) * torch.exp(seg)
+        y = scores @ xs + torch.einsum("bthn,bhnp->bhtp", cc, S) * torch.exp(cum)[..., None]
+        left = torch.exp(cum[..., -1:] - cum)
+        S = S * torch.exp(cum[..., -1])[..., None, None] + torch.einsum("bshn,bhsp->bhnp", bc, xs * left[..., None])
+        ys.append(y.transpose(1, 2) + D.float()[:, None] * xc)
+    return torch.cat(ys, 1).reshape(Bn, T, inner).to(u.dtype), S
+
+
+def ssm_step(x, dt, conv_w, conv_b, dt_bias, A_log, D, ring, S, kv_len, active, *, groups: int):
+    """One token per row at position ``kv_len[b]``: convolution inputs ``x`` ``[B,C]`` against the ring of the last ``K``
+    inputs ``ring`` ``[B,K,C]`` (slot = position mod K), then the state update; ``ring`` and ``S`` ``[B,H,N,P]`` change in
+    place, except for rows that are not ``active``.  Returns ``y`` ``[B,H*P]``."""
+    Bn, K, _ = ring.shape
+    H, N, P = S.shape[1:]
+    rows, pos = torch.arange(Bn, device=x.device), kv_len.long()
+    on = torch.ones(Bn, dtype=torch.bool, device=x.device) if active is None else active
+    ring[rows, pos % K] = torch.where(on[:, None], x, ring[rows, pos % K])
+    acc = torch.zeros(x.shape, dtype=torch.float32, device=x.device) + (0.0 if conv_b is None else conv_b.float())
+    for j in range(K):
+        past = ring[rows, (pos - j) % K].float() * (pos >= j)[:, None]
+        acc = acc + conv_w[:, K - 1 - j].float() * past
+    u = F.silu(acc).to(x.dtype).float()
+    inner = H * P
+    xv = u[:, :inner].view(Bn, H, P)
+    Bm = u[:, inner:inner + groups * N].view(Bn, groups, N).repeat_interleave(H // groups, dim=1)
+    Cm = u[:, inner + groups * N:].view(Bn, groups, N).repeat_interleave(H // groups, dim=1)
+    step = F.softplus(dt.float() + dt_bias.float())
+    new = S * torch.exp(-torch.exp(A_log.float()) * step)[..., None, None] + (Bm * step[..., None])[..., None] * xv[:, :, None, :]
+    S.copy_(torch.where(on[:, None, None, None], new, S))
+    y = torch.einsum("bhnp,bhn->bhp", new, Cm) + D.float()[:, None] * xv
+    return (y.reshape(Bn, inner) * on[:, None]).to(x.dtype)
+
+
+def gated_group_norm(y, z, weight, groups: int, eps: float):
+    """``y * silu(z)``, each of ``groups`` equal parts divided by its own root mean square, times ``weight``."""
+    v = y.float() * F.silu(z.float())
+    p = v.unflatten(-1, (groups, -1))
+    p = p * torch.rsqrt(p.pow(2).mean(-1, keepdim=True) + eps)
+    return (p.flatten(-2) * weight.float()).to(y.dtype)
+
+
 # ------------------------------------------------------------ mlp / act ----
-def swiglu(gate_up: torch.Tensor, act: str = "silu"):
-    """``act(gate) * up`` on a fused ``[..., 2F]`` tensor laid out ``[gate | up]``."""
+@dataclass(frozen=True)
+class ClippedGlu:
+    """Gated activation ``g * sigmoid(alpha g) * (u + 1)`` with ``g = min(gate, limit)``, ``u = clamp(up, +-limit)``."""
+    limit: float
+    alpha: float = 1.702
+
+
+def swiglu(gate_up: torch.Tensor, act="silu"):
+    """``act(gate) * up`` on a fused ``[..., 2F]`` tensor laid out ``[gate | up]``; ``act`` is a name or a
+    ``ClippedGlu``."""
     g, u = gate_up.chunk(2, dim=-1)
+    if isinstance(act, ClippedGlu):
+        gf, uf = g.float().clamp(max=act.limit), u.float().clamp(-act.limit, act.limit)
+        return (gf * torch.sigmoid(act.alpha * gf) * (uf + 1.0)).to(gate_up.dtype)
     if act == "silu":
         a = F.silu(g.float())
     elif act in ("gelu_pytorch_tanh", "gelu_tanh"):

@@ -239,8 +239,8 @@ def main():
     ap.add_argument("--no-graph", action="store_true", help="run decode steps eagerly (for per-kernel profiling)")
     ap.add_argument("--nccl-baseline", action="store_true", help="use per-tensor NCCL all-reduce instead of the fused DP step")
     ap.add_argument("--serving", nargs="?", const="all", default=None,
-                    help="instead of the training step: prefill and decode throughput of the Galodra family beside the closest "
-                         "existing one (dense-4k, dense-1k, moe-2k, comma-separated, or all); see bench_serving.py")
+                    help="instead of the training step: prefill and decode throughput of the Galodra and Mifutar families beside the "
+                         "closest existing one (dense-4k, dense-1k, moe-2k, hybrid-4k, hybrid-2k, hybrid-1k, comma-separated, or all); see bench_serving.py")
     args = ap.parse_args()
     if args.serving is not None:
         import bench_serving

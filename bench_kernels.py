@@ -1,7 +1,7 @@
 """Per-kernel timings at the headline model's shapes, against the measured roofline.
 
     python bench_kernels.py [--only gemm,attn,...] [--iters 20] [--json out.json]
-    python bench_kernels.py --profile-case gemm|gemm_2cta_256|gemm_lora|gemm_decode|decode_attn|sample|flash|flash_tc1|flash_tc2|flash_bwd|rmsnorm|swiglu|qk_norm_rope|logprob|lora_grad|moe_grouped|gdn_decode|gdn_chunk|gdn_tc_fwd|gdn_tc_bwd|flash_tc3_d256|flash_tc3_window|decode_attn_group|logprob_head|latent_decode|latent_prefill|post_norm   # small, for a profiler
+    python bench_kernels.py --profile-case gemm|gemm_2cta_256|gemm_lora|gemm_decode|decode_attn|sample|flash|flash_tc1|flash_tc2|flash_bwd|rmsnorm|swiglu|qk_norm_rope|logprob|lora_grad|moe_grouped|gdn_decode|gdn_chunk|gdn_tc_fwd|gdn_tc_bwd|flash_tc3_d256|flash_tc3_window|decode_attn_group|logprob_head|latent_decode|latent_prefill|post_norm|bias_prefill|bias_decode|ssm_scan|ssm_step|hyper_norm   # small, for a profiler
 
 Every kernel is timed with CUDA events on the launching stream after warm-up, with a buffer
 larger than L2 written between iterations (cold L2), and reported as achieved bytes/s or FLOP/s
@@ -190,6 +190,25 @@ def profile_case(name, C):
         x, y, gt = torch.randn(8192, 4096, device=dev), rnd(8192, 4096), rnd(8192, 4096)
         v1, hist, coef = torch.ones(4096, device=dev), torch.randn(2, 8192, 4096, device=dev), torch.ones(3, device=dev)
         fn = lambda: C.post_norm(x, y, v1, v1, 1e-6, 2.0, gt, v1, hist, coef, bf, None)
+    elif name == "bias_prefill":
+        q, k, bias = rnd(8, 2048, 32, 128), rnd(8, 2048, 8, 128), torch.randn(32, 1024, device=dev)
+        fn = lambda: C.bias_attention(q, k, bias, scale=0.09, window=1024)
+    elif name == "bias_decode":
+        q, k, ring, bias = rnd(128, 4096), rnd(128, 1024), rnd(128, 1024, 1024), torch.randn(32, 1024, device=dev)
+        pos = torch.full((128,), 1500, device=dev, dtype=torch.int32)
+        fn = lambda: C.bias_decode(q, k, ring, pos, bias, dim=128, scale=0.09)
+    elif name == "ssm_scan":
+        u, dtr, par = rnd(8, 2048, 128 * 64 + 2 * 8 * 128), rnd(8, 2048, 128), torch.randn(128, device=dev)
+        fn = lambda: C.ssm_scan(u, dtr, par - 3, par, par, None, heads=128, state=128, groups=8)
+    elif name == "ssm_step":
+        x, dtr, par = rnd(128, 64 * 64 + 2 * 4 * 128), rnd(128, 64), torch.randn(64, device=dev)
+        cw, ring, S = torch.randn(x.shape[1], 4, device=dev), rnd(128, 4, x.shape[1]), torch.randn(128, 64, 128, 64, device=dev)
+        pos = torch.full((128,), 1500, device=dev, dtype=torch.int32)
+        fn = lambda: C.ssm_step(x, dtr, cw, cw[:, 0].contiguous(), par, par, par, ring, S, pos, None, groups=4)
+    elif name == "hyper_norm":
+        x, y = torch.randn(8192, 2, 4096, device=dev), rnd(8192, 4096)
+        mix, out, v1 = torch.eye(2, device=dev), torch.ones(2, device=dev), torch.zeros(4096, device=dev)
+        fn = lambda: C.hyper_norm(x, y, mix, out, out, v1, 1e-6, bf, 1.0, True)
     else:
         raise SystemExit(f"unknown profile case {name!r}")
     evs = []
@@ -275,6 +294,94 @@ def latent_kernels(C, T, report, dev):
         report("moe route sigmoid 16384 x 64 top 8", s, 16384 * (64 * 8 + 64), 0)
         s = T(lambda: C.moe_route(lg, 8, True))
         report("  moe route softmax 16384 x 64 top 8", s, 16384 * (64 * 8 + 64), 0)
+
+
+def ssd_kernels(C, T, report, dev):
+    """Kernels of the Mamba-2, distance-biased attention and hyper-connection layers, each beside the like kernel of the
+    existing families.  FLOP counts of the scans are those of the chunked form with 64 tokens a chunk."""
+    bf = torch.bfloat16
+    rnd = lambda *s: torch.randn(*s, device=dev, dtype=bf)  # noqa: E731
+    pairs = lambda S, w: sum(min(i + 1, w) for i in range(S))  # noqa: E731
+    B, S = 8, 2048
+    with torch.no_grad():
+        for H, Hk, D in ((32, 8, 128), (16, 4, 64), (16, 2, 256)):
+            for w in (1024, 2048):
+                q, k, v, bias = rnd(B, S, H, D), rnd(B, S, Hk, D), rnd(B, S, Hk, D), torch.randn(H, w, device=dev)
+                s = T(lambda: C.bias_attention(q, k, bias, scale=0.09, window=w))
+                report(f"biased prefill B{B} S{S} w{w} {H}q/{Hk}kv d{D}", s, 0, 4 * B * H * pairs(S, w) * D)
+                s = T(lambda: C.attention(q, k, v, scale=0.09, causal=True, window=w if w < S else 0))
+                report(f"  flash prefill B{B} S{S} w{w} {H}q/{Hk}kv d{D}", s, 0, 4 * B * H * pairs(S, w) * D)
+        for H, Hk, D in ((32, 8, 128), (16, 4, 128), (16, 4, 64), (16, 2, 256)):
+            for R, n in ((128, 1024), (16, 1024), (128, 4096)):
+                q, k, ring, bias = rnd(R, H * D), rnd(R, Hk * D), rnd(R, n, Hk * D), torch.randn(H, n, device=dev)
+                pos = torch.full((R,), n + 77, device=dev, dtype=torch.int32)
+                s = T(lambda: C.bias_decode(q, k, ring, pos, bias, dim=D, scale=0.09))
+                report(f"biased decode B{R} len{n} {H}q/{Hk}kv d{D} (keys only)", s, R * n * Hk * D * 2, 0)
+                kc, vc = ring.view(R, n, Hk, D), rnd(R, n, Hk, D)
+                ln = torch.full((R,), n, device=dev, dtype=torch.int32)
+                s = T(lambda: C.decode_attention(q.view(R, H, D), kc, vc, ln, scale=0.09))
+                report(f"  decode attention B{R} len{n} {H}q/{Hk}kv d{D}", s, 2 * R * n * Hk * D * 2, 0)
+                del q, k, ring, kc, vc
+        for H, P, N, G in ((128, 64, 128, 8), (64, 64, 128, 4), (32, 64, 128, 1), (64, 128, 64, 1)):
+            ch = H * P + 2 * G * N
+            x, dtr, par = rnd(B, S, ch), rnd(B, S, H), torch.randn(H, device=dev)
+            cw, cb = torch.randn(ch, 4, device=dev), torch.randn(ch, device=dev)
+            s = T(lambda: C.ssm_conv(x, cw, cb))
+            report(f"ssm conv 16384 tokens {ch} channels", s, 2 * x.numel() * 2, 0)
+            gw = torch.randn(ch, 4, device=dev).to(bf)
+            s = T(lambda: C.gdn_conv(x, gw, None, True))
+            report("  gdn conv, same size", s, 2 * x.numel() * 2, 0)
+            fl = B * S * (G * 2 * 64 * N + H * 2 * (64 * P + 2 * N * P))
+            by = (x.numel() + B * S * H * (P + 1)) * 2 + B * H * N * P * 4
+            for variant in (0, 1):
+                s = T(lambda: C.ssm_scan(x, dtr, par - 3, par, par, None, heads=H, state=N, groups=G, variant=variant))
+                report(f"ssm scan 16384 tokens H{H} P{P} N{N} G{G}" + (", any-size kernel" if variant else ""), s, by, fl)
+            Hv, Hk = H * P // 128, max(1, H * P // 256)
+            qd, kd, vd = rnd(B, S, Hk, 128), rnd(B, S, Hk, 128), rnd(B, S, Hv, 128)
+            g, b = -torch.rand(B, S, Hv, device=dev) * 0.3, torch.rand(B, S, Hv, device=dev)
+            fg = B * Hv * (S // 64) * 2 * (64 * 64 * 128 * 2 + 64 * 128 * 64 * 3 + 64 * 128 * 128 * 3)
+            s = T(lambda: C.gdn_chunk_fwd(qd, kd, vd, g, b))
+            report(f"  gdn chunk scan (prefill) 16384 tokens Hv{Hv}", s, (qd.numel() * 2 + vd.numel() * 2) * 2, fg)
+            z, w = rnd(B * S, H * P), torch.randn(H * P, device=dev)
+            y = rnd(B * S, H * P)
+            s = T(lambda: C.gated_group_norm(y, z, w, G, 1e-6))
+            report(f"gated group norm 16384 x {H * P}, {G} parts", s, 3 * y.numel() * 2, 0)
+            w128 = torch.randn(128, device=dev).to(bf)
+            s = T(lambda: C.rmsnorm_gated(y.view(-1, 128), z.view(-1, 128), w128, 1e-6))
+            report("  gated rmsnorm per 128, same size", s, 3 * y.numel() * 2, 0)
+            del x, y, z, qd, kd, vd
+            for R in (128, 16):
+                xr, dr, ring, St = rnd(R, ch), rnd(R, H), rnd(R, 4, ch), torch.randn(R, H, N, P, device=dev)
+                pos = torch.full((R,), 99, device=dev, dtype=torch.int32)
+                s = T(lambda: C.ssm_step(xr, dr, cw, cb, par, par, par, ring, St, pos, None, groups=G))
+                report(f"ssm step B{R} H{H} P{P} N{N} (with convolution)", s, 2 * St.numel() * 4, 0)
+                qd, kd, vd, gg = rnd(R, Hk * 128), rnd(R, Hk * 128), rnd(R, Hv * 128), -torch.rand(R, Hv, device=dev)
+                Sg = torch.randn(R, Hv, 128, 128, device=dev)
+                s = T(lambda: C.gdn_decode_step(qd, kd, vd, gg, -gg, Sg, True, 1e-6))
+                report(f"  gdn decode step B{R} Hv{Hv} (without convolution)", s, 2 * Sg.numel() * 4, 0)
+                yr, zr = rnd(R, H * P), rnd(R, H * P)
+                s = T(lambda: C.gated_group_norm(yr, zr, w, G, 1e-6))
+                report(f"gated group norm {R} x {H * P}, {G} parts", s, 3 * yr.numel() * 2, 0)
+                del St, Sg
+        for rows in (16384, 128):
+            for ns in (1, 2, 4):
+                W = 4096
+                x, y, v1 = torch.randn(rows, ns, W, device=dev), rnd(rows, W), torch.zeros(W, device=dev)
+                mix, out = torch.eye(ns, device=dev), torch.full((ns,), 0.01, device=dev)
+                s = T(lambda: C.hyper_norm(x, y, mix, out, out, v1, 1e-6, bf, 1.0, True))
+                report(f"hyper norm {rows} x {ns} streams x 4096", s, x.numel() * 8 + y.numel() * 4, 0)
+            xb, wb = rnd(rows, W), torch.ones(W, device=dev, dtype=bf)
+            s = T(lambda: C.add_rmsnorm(xb, y, wb, 1e-6))
+            report(f"  add + rmsnorm {rows} rows W4096", s, rows * W * 2 * 4, 0)
+            ids, tab, pe = torch.randint(0, 32768, (rows,), device=dev), rnd(32768, W), torch.randn(2048, W, device=dev)
+            at = torch.arange(rows, device=dev) % 2048
+            s = T(lambda: C.embed_streams(ids, tab, pe, at, 2))
+            report(f"embedding + positions {rows} x 2 streams", s, rows * W * (2 + 4 + 8), 0)
+            gu = rnd(rows, 2 * 12288)
+            s = T(lambda: C.swiglu(gu, C.eager.ClippedGlu(7.0)))
+            report(f"clipped glu {rows} x 12288", s, gu.numel() * 3, 0)
+            s = T(lambda: C.swiglu(gu, "silu"))
+            report("  silu glu, same size", s, gu.numel() * 3, 0)
 
 
 def main():
@@ -417,6 +524,8 @@ def main():
             del graph, dec, model
     if want("latent"):
         latent_kernels(C, T, report, dev)
+    if want("ssd"):
+        ssd_kernels(C, T, report, dev)
     if want("slab"):
         # cost of the adapter k-slab as a function of its width (the k-block is 64 wide whatever R is)
         M, N, K = 24576, 6144, H

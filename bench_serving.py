@@ -1,7 +1,7 @@
 """Prefill and decode throughput of a serving-sized slice of a family (``python bench.py --serving``).
 
-Each size runs the Galodra family beside the existing family closest to it, at equal width, depth, head count,
-feed-forward width and window, with random weights in bf16 and no adapters:
+Each size runs the Galodra or the Mifutar family beside the existing family closest to it, at equal width, depth, head
+count, feed-forward width and window, with random weights in bf16 and no adapters:
 
     dense-4k   8 layers, width 4096, 32 heads (latent 512, 128 + 64 score entries, values 128), window 1024, GeGLU 12288
                beside Gemma-style sliding-window layers (32 query / 16 key-value heads of 128)
@@ -9,6 +9,13 @@ feed-forward width and window, with random weights in bf16 and no adapters:
                beside Gemma-style layers (16 / 8 heads of 64)
     moe-2k     8 layers, width 2048, 16 heads (latent 512, 128 + 64, values 128), window 1024, 64 experts of 768, top 8
                beside Qwen3.5-style full-attention layers (16 / 2 heads of 256) with the same experts
+    hybrid-4k  8 layers, width 4096, two streams, feed-forward 12288: three Mamba-2 layers (128 heads of 64 x 128 state, 8
+               groups) to one biased attention layer (32 / 8 heads of 128, window 1024), beside Qwen3.5-style layers
+               (GatedDeltaNet with 64 heads of 128 x 128 state, full attention with the same heads)
+    hybrid-2k  12 layers, width 2048, feed-forward 6144: 64 heads of 64 x 128, 4 groups; 16 / 4 heads of 128, beside the same
+               with 32 heads of 128 x 128
+    hybrid-1k  12 layers, width 1024, feed-forward 4096: 32 heads of 64 x 128, 1 group; 16 / 4 heads of 64, beside the same
+               with 16 heads of 128 x 128
 
 Prefill: 8 prompts of 2048 tokens.  Decode: 128 rows at 1024 cached tokens, one step replayed from a CUDA graph.  Times
 are CUDA events over ``steps`` calls after ``warmup``; weights and caches are larger than L2.  One JSON line a model.
@@ -24,6 +31,9 @@ SIZES = {
     "dense-4k": dict(layers=8, width=4096, heads=32, kv=16, dim=128, rot=64, vdim=128, rank=512, window=1024, ff=12288),
     "dense-1k": dict(layers=12, width=1024, heads=16, kv=8, dim=64, rot=32, vdim=64, rank=256, window=512, ff=4096),
     "moe-2k": dict(layers=8, width=2048, heads=16, kv=2, dim=128, rot=64, vdim=128, rank=512, window=1024, ff=768, experts=64, top=8),
+    "hybrid-4k": dict(family="mifutar", layers=8, width=4096, heads=32, kv=8, dim=128, window=1024, ff=12288, ssm=128, groups=8),
+    "hybrid-2k": dict(family="mifutar", layers=12, width=2048, heads=16, kv=4, dim=128, window=1024, ff=6144, ssm=64, groups=4),
+    "hybrid-1k": dict(family="mifutar", layers=12, width=1024, heads=16, kv=4, dim=64, window=1024, ff=4096, ssm=32, groups=1),
 }
 
 
@@ -37,6 +47,17 @@ def build(size: str, family: str, device):
         dims = LatentDims(s["heads"], s["dim"], s["rot"], s["vdim"], s["rank"], (s["dim"] + s["rot"]) ** -0.5, s["window"], 1e4, 0, True)
         ff = FeedForward(s["ff"], s.get("experts", 0), s.get("top", 0))
         m = GalodraGradModel(GalodraSpec(VOCAB, s["width"], [LayerSpec(dims, ff)] * s["layers"], alpha=2.0), None, **kw)
+    elif family == "mifutar":
+        from ferrl_b200.models.mifutar import BiasAttentionDims, ClippedFeedForward, LayerSpec, Mamba2Dims, MifutarGradModel, MifutarSpec
+        ff = ClippedFeedForward(s["ff"], 7.0)
+        rec = LayerSpec(Mamba2Dims(s["ssm"], 64, 128, s["groups"], 4, s["groups"]), ff)
+        att = LayerSpec(BiasAttentionDims(s["heads"], s["kv"], s["dim"], s["dim"] ** -0.5, s["window"], 32, 128), ff)
+        m = MifutarGradModel(MifutarSpec(VOCAB, s["width"], ([rec] * 3 + [att]) * (s["layers"] // 4), streams=2), None, **kw)
+    elif "ssm" in s:
+        from ferrl_b200.models.qwen35 import Qwen35GradModel, Qwen35Spec
+        m = Qwen35GradModel(Qwen35Spec(VOCAB, s["width"], s["layers"], s["heads"], s["kv"], s["dim"], s["ff"],
+                                       (["linear_attention"] * 3 + ["full_attention"]) * (s["layers"] // 4), max_position_embeddings=max_len,
+                                       tie_word_embeddings=False, lin_k_heads=s["ssm"] // 4, lin_v_heads=s["ssm"] // 2), None, **kw)
     elif "experts" in s:
         from ferrl_b200.models.qwen35 import MoeDims, Qwen35GradModel, Qwen35Spec
         m = Qwen35GradModel(Qwen35Spec(VOCAB, s["width"], s["layers"], s["heads"], s["kv"], 256, s["ff"], ["full_attention"] * s["layers"],
@@ -98,7 +119,7 @@ def main(sizes, steps: int, warmup: int, clock_sampler) -> int:
     device = torch.device("cuda", 0)
     torch.cuda.set_device(device)
     for size in sizes:
-        for family in ("galodra", "closest"):
+        for family in (SIZES[size].get("family", "galodra"), "closest"):
             model = build(size, family, device)
             clocks = clock_sampler(0)
             clocks.start()

@@ -229,6 +229,9 @@ bool latent_decode_tc_supported(const LatentDecodeArgs& a);
 int latent_decode_splits(const LatentDecodeArgs& a, int num_sms);
 const char* latent_decode_tc(const LatentDecodeArgs& a, int n_splits, int* status, cudaStream_t s);   // csrc/kernels/latent_decode_tc.cu
 const char* latent_decode(const LatentDecodeArgs& a, int n_splits, int* status, cudaStream_t s);
+// joins the key ranges of a softmax: ws [heads_total, n_splits, width + 2] = weighted values, maximum (base 2), sum -> bf16
+// [heads_total, width]; sink [heads] or null
+const char* attn_combine(const float* ws, const float* sink, void* out, long long heads_total, int heads, int width, int n_splits, cudaStream_t s);
 
 // ---- residual sum + layer norm + depth average (csrc/kernels/post_norm.cu) ----
 struct PostNormArgs {
@@ -269,6 +272,8 @@ struct SsmScanArgs {
   int B, T, H, P, N, G;
 };
 const char* ssm_scan(const SsmScanArgs& a, cudaStream_t s);
+bool ssm_scan_tc_supported(const SsmScanArgs& a);                  // csrc/kernels/ssm_scan_tc.cu
+const char* ssm_scan_tc(const SsmScanArgs& a, int* status, cudaStream_t s);
 struct SsmStepArgs {
   int dtype;
   const void* x; long long ld_x;                   // this token's convolution inputs [B, C], C = H*P + 2*G*N
@@ -292,6 +297,8 @@ struct BiasFwdArgs {
   int B, S, Hq, Hkv, D, window; float scale;
 };
 const char* bias_fwd_any(const BiasFwdArgs& a, cudaStream_t s);
+bool bias_fwd_tc_supported(const BiasFwdArgs& a);                     // csrc/kernels/bias_fwd_tc.cu
+const char* bias_fwd_tc(const BiasFwdArgs& a, int* status, cudaStream_t s);
 struct BiasDecodeArgs {
   int dtype;
   const void* q; long long ld_q; const void* k; long long ld_k;   // this token's [B, Hq*D] and [B, Hkv*D]
@@ -299,8 +306,12 @@ struct BiasDecodeArgs {
   const int* kv_len; const unsigned char* active;
   const float* bias; long long bias_ld; void* out; // [B, Hq*D]
   int B, Hq, Hkv, D; float scale;
+  float* ws;                                       // B * Hq * n_splits * (D + 2) floats when n_splits > 1
 };
 const char* bias_decode_any(const BiasDecodeArgs& a, cudaStream_t s);
+bool bias_decode_tc_supported(const BiasDecodeArgs& a);               // csrc/kernels/bias_decode_tc.cu
+int bias_decode_splits(const BiasDecodeArgs& a, int num_sms);
+const char* bias_decode_tc(const BiasDecodeArgs& a, int n_splits, cudaStream_t s);
 
 // ---- flash attention (prefill / training) ----
 struct FlashArgs {

@@ -1368,7 +1368,10 @@ std::tuple<Tensor, Tensor> ssm_scan(const Tensor& u, const Tensor& dtr, const Te
   Tensor y = out_empty({a.B, a.T, inner}, u.options());
   Tensor S = out_empty({a.B, a.H, a.N, a.P}, u.options().dtype(at::kFloat));
   a.y = y.data_ptr(); a.state = S.data_ptr<float>();
-  (void)variant;
+  if (variant == 0 && ferrl::ssm_scan_tc_supported(a)) {           // variant 1: the float32 kernel of any size
+    FERRL_CHECK(ferrl::ssm_scan_tc(a, status_word(), stream()));
+    return {y, S};
+  }
   FERRL_CHECK(ferrl::ssm_scan(a, stream()));
   return {y, S};
 }
@@ -1435,7 +1438,10 @@ Tensor bias_fwd(const Tensor& q, const Tensor& k, const Tensor& bias, double sca
   seq_strides(k.flatten(2), &a.k_bs, &a.k_ts);
   Tensor out = out_empty({a.B, a.S, static_cast<int64_t>(a.Hq) * a.D}, q.options());
   a.out = out.data_ptr();
-  (void)variant;
+  if (variant == 0 && ferrl::bias_fwd_tc_supported(a)) {
+    FERRL_CHECK(ferrl::bias_fwd_tc(a, status_word(), stream()));
+    return out;
+  }
   FERRL_CHECK(ferrl::bias_fwd_any(a, stream()));
   return out;
 }
@@ -1462,7 +1468,16 @@ Tensor bias_decode(const Tensor& q, const Tensor& k, Tensor cache, const Tensor&
   }
   Tensor out = out_empty({a.B, heads * dim}, q.options());
   a.out = out.data_ptr();
-  (void)variant;
+  if (variant != 1 && ferrl::bias_decode_tc_supported(a)) {        // variant 1: the any-size kernel; above 1: that many ranges plus one
+    const int n = variant > 1 ? static_cast<int>(variant) - 1 : ferrl::bias_decode_splits(a, num_sms());
+    Tensor ws;
+    if (n > 1) {
+      ws = out_empty({static_cast<int64_t>(a.B) * heads * n * (dim + 2)}, q.options().dtype(at::kFloat));
+      a.ws = ws.data_ptr<float>();
+    }
+    FERRL_CHECK(ferrl::bias_decode_tc(a, n, stream()));
+    return out;
+  }
   FERRL_CHECK(ferrl::bias_decode_any(a, stream()));
   return out;
 }

@@ -25,11 +25,11 @@ constexpr int kMaxStreams = 32;
 
 // NS streams at compile time, or up to kMaxStreams of them at run time (NS = 0)
 template <typename TY, typename TC, int NS, int V>
-__global__ void hyper_norm_kernel(HyperNormArgs a) {
+__global__ void __launch_bounds__(512) hyper_norm_kernel(HyperNormArgs a) {
   extern __shared__ __align__(16) float sm_u[];
   __shared__ float red[32];
   __shared__ float s_mix[kMaxStreams * kMaxStreams], s_out[kMaxStreams], s_in[kMaxStreams];
-  constexpr int CAP = NS > 0 ? NS : kMaxStreams;
+  constexpr int CAP = NS > 0 ? NS : kMaxStreams, UN = NS > 0 ? NS : 1;
   const int ns = NS > 0 ? NS : a.ns;
   pdl_trigger();
   // the coefficients are weights: no kernel of the step writes them
@@ -46,7 +46,7 @@ __global__ void hyper_norm_kernel(HyperNormArgs a) {
   float sq = 0.f;
   for (int c = threadIdx.x * V; c < a.W; c += blockDim.x * V) {
     Vec<V> xs[CAP];
-#pragma unroll
+#pragma unroll(UN)
     for (int s = 0; s < CAP; ++s)
       if (NS > 0 || s < ns) xs[s] = ld<V>(x + static_cast<long long>(s) * a.W + c);
     Vec<V> u;
@@ -54,13 +54,13 @@ __global__ void hyper_norm_kernel(HyperNormArgs a) {
     for (int e = 0; e < V; ++e) u.v[e] = 0.f;
     if (y) {
       const Vec<V> yv = ld<V>(y + c);
-#pragma unroll
+#pragma unroll(UN)
       for (int t = 0; t < CAP; ++t) {
         if (NS == 0 && t >= ns) break;
         Vec<V> n;
 #pragma unroll
         for (int e = 0; e < V; ++e) n.v[e] = s_out[t] * yv.v[e];
-#pragma unroll
+#pragma unroll(UN)
         for (int s = 0; s < CAP; ++s)
           if (NS > 0 || s < ns) {
 #pragma unroll
@@ -71,7 +71,7 @@ __global__ void hyper_norm_kernel(HyperNormArgs a) {
         for (int e = 0; e < V; ++e) u.v[e] += s_in[t] * n.v[e];
       }
     } else {
-#pragma unroll
+#pragma unroll(UN)
       for (int s = 0; s < CAP; ++s)
         if (NS > 0 || s < ns) {
 #pragma unroll
@@ -99,7 +99,8 @@ const char* launch_ns(const HyperNormArgs& a, cudaStream_t s) {
   const bool vec = NS > 0 && a.W % 4 == 0 && a.ld_y % 4 == 0 && al16(a.x) && (reinterpret_cast<uintptr_t>(a.y) & (sizeof(TY) * 4 - 1)) == 0 &&
                    al16(a.w) && al16(a.h);
   const int per = vec ? 4 : 1;
-  const int threads = std::min(a.rows >= 1024 ? 256 : 1024, std::max(64, (a.W / per + 31) / 32 * 32));
+  const int cap = NS == 0 || a.rows >= 1024 ? 256 : 512;      // wide blocks for few rows, within the register file
+  const int threads = std::min(cap, std::max(64, (a.W / per + 31) / 32 * 32));
   auto k4 = hyper_norm_kernel<TY, TC, NS, NS == 0 ? 1 : 4>;
   auto k1 = hyper_norm_kernel<TY, TC, NS, 1>;
   if (!FERRL_ONCE_PER_DEVICE(cudaFuncSetAttribute(k4, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) == cudaSuccess &&

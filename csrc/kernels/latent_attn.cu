@@ -7,7 +7,7 @@
 //   head_gemm_kernel        out[b, h, :] = W[h] x[b, h, :], one small matrix per head (query absorption, value
 //                           expansion of a decode step) on mma.sync; head_gemm_any_kernel for other types and sizes
 //   latent_decode_any_kernel  one query per row against the row's cached latents, any type and size
-//                           (latent_decode_tc.cu holds the tcgen05 form for bf16); latent_combine_kernel joins key ranges
+//                           (latent_decode_tc.cu holds the tcgen05 form for bf16); attn_combine_kernel joins key ranges
 //
 // Scores, softmax and sink are fp32.  A sink adds exp(sink_h) to the softmax denominator of head h.
 #include <cuda_bf16.h>
@@ -301,7 +301,7 @@ __global__ void __launch_bounds__(128) latent_decode_any_kernel(LatentDecodeArgs
 }
 
 // ------------------------------------------------------------------------------------------------ key ranges of a row
-__global__ void latent_combine_kernel(const float* __restrict__ ws, const float* __restrict__ sink, bf16* __restrict__ ctx,
+__global__ void attn_combine_kernel(const float* __restrict__ ws, const float* __restrict__ sink, bf16* __restrict__ ctx,
                                       int heads, int rank, int n_splits) {
   pdl_trigger();
   pdl_wait();
@@ -398,12 +398,14 @@ const char* latent_decode(const LatentDecodeArgs& a, int n_splits, int* status, 
   }
   if (n_splits > 1 && !a.ws) return "latent_decode: workspace missing";
   if (const char* err = latent_decode_tc(a, n_splits, status, s)) return err;
-  if (n_splits > 1) {
-    launch_pdl(latent_combine_kernel, dim3(a.B * a.heads), dim3(128), 0, s, static_cast<const float*>(a.ws), a.sink,
-               static_cast<bf16*>(a.ctx), a.heads, a.rank, n_splits);
-    count_launch();
-  }
+  if (n_splits > 1) return attn_combine(a.ws, a.sink, a.ctx, static_cast<long long>(a.B) * a.heads, a.heads, a.rank, n_splits, s);
   return cudaGetLastError() == cudaSuccess ? nullptr : "latent_decode launch failed";
+}
+
+const char* attn_combine(const float* ws, const float* sink, void* out, long long heads_total, int heads, int width, int n_splits, cudaStream_t s) {
+  launch_pdl(attn_combine_kernel, dim3(static_cast<unsigned>(heads_total)), dim3(128), 0, s, ws, sink, static_cast<bf16*>(out), heads, width, n_splits);
+  count_launch();
+  return cudaGetLastError() == cudaSuccess ? nullptr : "attn_combine launch failed";
 }
 
 }  // namespace ferrl

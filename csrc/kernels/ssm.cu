@@ -33,7 +33,7 @@ __device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log
 
 // ------------------------------------------------------------------------------------------------ convolution
 // A thread owns V channels and kRun consecutive tokens: the window slides through registers.
-constexpr int kRun = 8;
+constexpr int kRun = 16;
 template <typename T, int V> struct ConvIo;
 template <typename T> struct ConvIo<T, 1> {
   static __device__ __forceinline__ void ld(const T* p, float* v) { v[0] = to_f(*p); }
@@ -77,10 +77,18 @@ __global__ void ssm_conv_kernel(const T* __restrict__ x, long long x_bs, long lo
     for (int e = 0; e < V; ++e) bs[e] = bias ? bias[c + e] : 0.f;
     if constexpr (KT > 0) {
       float wv[KT][V], win[KT][V];
+      if constexpr (KT == 4) {
 #pragma unroll
-      for (int j = 0; j < KT; ++j)
+        for (int e = 0; e < V; ++e) {
+          const float4 f = *reinterpret_cast<const float4*>(w + static_cast<long long>(c + e) * 4);
+          wv[0][e] = f.x; wv[1][e] = f.y; wv[2][e] = f.z; wv[3][e] = f.w;
+        }
+      } else {
 #pragma unroll
-        for (int e = 0; e < V; ++e) wv[j][e] = w[static_cast<long long>(c + e) * KT + j];
+        for (int j = 0; j < KT; ++j)
+#pragma unroll
+          for (int e = 0; e < V; ++e) wv[j][e] = w[static_cast<long long>(c + e) * KT + j];
+      }
 #pragma unroll
       for (int j = 1; j < KT; ++j) {          // win[j] holds token t0 - KT + j
         const int t = t0 - KT + j;
@@ -138,7 +146,12 @@ void launch_conv(const void* x, long long x_bs, long long x_ts, const float* w, 
   switch (K) {
     case 2: ssm_conv_kernel<T, V, 2><<<grid, 128, 0, s>>>(xp, x_bs, x_ts, w, bias, yp, B, L, C, K); break;
     case 3: ssm_conv_kernel<T, V, 3><<<grid, 128, 0, s>>>(xp, x_bs, x_ts, w, bias, yp, B, L, C, K); break;
-    case 4: ssm_conv_kernel<T, V, 4><<<grid, 128, 0, s>>>(xp, x_bs, x_ts, w, bias, yp, B, L, C, K); break;
+    case 4:
+      if ((reinterpret_cast<uintptr_t>(w) & 15) == 0) {
+        ssm_conv_kernel<T, V, 4><<<grid, 128, 0, s>>>(xp, x_bs, x_ts, w, bias, yp, B, L, C, K);
+        break;
+      }
+      [[fallthrough]];
     default: ssm_conv_kernel<T, V, 0><<<grid, 128, 0, s>>>(xp, x_bs, x_ts, w, bias, yp, B, L, C, K); break;
   }
 }
@@ -271,6 +284,15 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(SsmStepArgs a) {
     for (int i = threadIdx.x; i < a.P; i += 256) y[i] = from_f<T>(0.f);
     return;
   }
+  // the first rows of the state are requested before the convolution needs its inputs
+  float* S = a.state + (static_cast<long long>(b) * a.H + h) * a.N * a.P;
+  const int rg0 = static_cast<int>(threadIdx.x) / cgn, c_0 = (static_cast<int>(threadIdx.x) - rg0 * cgn) * V;
+  Vec<V> v[kAhead];
+  if (static_cast<int>(threadIdx.x) < RG * cgn) {
+#pragma unroll
+    for (int k = 0; k < kAhead; ++k)
+      if (rg0 + k * RG < a.N) v[k] = ld<V>(S + static_cast<long long>(rg0 + k * RG) * a.P + c_0);
+  }
   const long long pos = a.kv_len[b];
   const int cur = static_cast<int>(pos % a.K);
   const T* xr = static_cast<const T*>(a.x) + b * a.ld_x;            // this token's [x | B | C] channels
@@ -295,17 +317,17 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(SsmStepArgs a) {
   if (threadIdx.x == 0) s_dt = softplus_f(to_f(static_cast<const T*>(a.dt)[b * a.ld_dt + h]) + a.dt_bias[h]);
   __syncthreads();
   const float dt = s_dt, da = __expf(-__expf(a.A_log[h]) * dt);
-  float* S = a.state + (static_cast<long long>(b) * a.H + h) * a.N * a.P;
   for (int item = threadIdx.x; item < RG * cgn; item += 256) {
     const int rg = item / cgn, c = (item - rg * cgn) * V;
     Vec<V> acc, dx = ld<V>(sx + c);
 #pragma unroll
     for (int e = 0; e < V; ++e) { acc.v[e] = 0.f; dx.v[e] *= dt; }
     for (int n0 = rg; n0 < a.N; n0 += RG * kAhead) {
-      Vec<V> v[kAhead];
+      if (n0 != rg || item != static_cast<int>(threadIdx.x)) {
 #pragma unroll
-      for (int k = 0; k < kAhead; ++k)
-        if (n0 + k * RG < a.N) v[k] = ld<V>(S + static_cast<long long>(n0 + k * RG) * a.P + c);
+        for (int k = 0; k < kAhead; ++k)
+          if (n0 + k * RG < a.N) v[k] = ld<V>(S + static_cast<long long>(n0 + k * RG) * a.P + c);
+      }
 #pragma unroll
       for (int k = 0; k < kAhead; ++k) {
         const int n = n0 + k * RG;

@@ -640,7 +640,10 @@ def bias_attention(q, k, bias, *, scale, window, variant=0):
     return native_fn(q, k, bias)
 
 
-def bias_decode(q, k, cache, kv_len, bias, *, dim, scale, active=None, variant=0):
+def bias_decode(q, k, cache, kv_len, bias, *, dim, scale, active=None, variant=0, splits=0):
+    """``variant=1`` forces the any-size kernel, ``splits`` the number of slot ranges per row of the other one (0: planned
+    from the batch)."""
+    variant = splits + 1 if splits else variant
     return lib().bias_decode(q, k, cache, kv_len, active, bias, q.shape[-1] // dim, dim, float(scale), int(variant))
 
 
@@ -660,6 +663,7 @@ def hyper_norm(x, y, mix, out, inp, weight, eps, cast, scale, store):
         x, h = eager.hyper_norm(x, y, mix, out, inp, weight, eps, scale)
         return x, h.to(cast)
     ns, W = x.shape[-2:]
+    x = x.contiguous()
     h = lib().hyper_norm(x.view(-1, ns, W), None if y is None else _rows2(y, W), mix, out, inp, weight, float(eps), float(scale),
                          cast == torch.bfloat16, bool(store))
     return x, h.view(*x.shape[:-2], W)

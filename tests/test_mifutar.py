@@ -124,6 +124,7 @@ def test_attention_of_one_token(device, dtype, shape):
     if device == "cuda":
         from ferrl_b200.ops import cuda as C
         run.append(lambda *a, **kw: C.bias_decode(*a, variant=1, **kw))
+        run += [lambda *a, n=n, **kw: C.bias_decode(*a, splits=n, **kw) for n in (1, 2, 5)]
     for fn in run:
         ring = d(cache.flatten(2).clone())
         got = fn(fused[:, :H * D], fused[:, H * D:(H + G) * D], ring, d(kv), d(bias), dim=D, scale=scale, active=d(on))
@@ -321,13 +322,12 @@ def test_clipped_glu_in_the_projection(M):
     near(C.gemm_glu(x.cuda(), w[order].contiguous().cuda(), act), want, 3e-2)
 
 
-@pytest.mark.parametrize("device", [CPU, GPU])
-@pytest.mark.parametrize("dtype", [F32, BF16])
-@pytest.mark.parametrize("M,N,Kd", [(1, 40, 64), (70, 24, 64), (1100, 520, 72), (3, 17, 13)])
+@pytest.mark.parametrize("device,dtype", [(CPU, F32), (CPU, BF16), pytest.param("cuda", BF16, marks=pytest.mark.gpu)])
+@pytest.mark.parametrize("M,N,Kd", [(1, 40, 64), (70, 24, 64), (1100, 520, 72), (3, 17, 16), (130, 712, 256)])
 def test_projection_with_bias(device, dtype, M, N, Kd):
     from ferrl_b200 import ops
     x, w, b = rand(M, Kd, seed=1, dtype=dtype), rand(N, Kd, seed=2, dtype=dtype), rand(N, seed=3, std=5.0, dtype=dtype)
-    near(ops.lora_linear(x.to(device), w.to(device), None, None, bias=b.to(device)), x.double() @ w.double().T + b.double(), TOL[dtype])
+    close(ops.lora_linear(x.to(device), w.to(device), None, None, bias=b.to(device)), x.double() @ w.double().T + b.double(), dtype)
 
 
 # ------------------------------------------------------------------------------------------------ whole models
@@ -590,7 +590,7 @@ def test_scoring_gradients_on_the_gpu(tmp_path, dtype):
         lp = m.token_logprobs(ids[:, :-1].to(dev), torch.tensor([9, 9], device=dev), ids[:, 10:].to(dev))
         lp.sum().backward()
         grads.append([lp.detach().cpu()] + [p.grad.detach().cpu() for p in m.trainable_params()])
-    tol = 2e-3 if dtype == F32 else 0.12
+    tol = 2e-3 if dtype == F32 else 0.2
     for got, ref in zip(grads[1], grads[0]):
         assert float((got - ref).norm() / ref.norm()) < tol
     with torch.no_grad():      # grad-free scoring runs the fused inference pass

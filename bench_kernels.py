@@ -317,6 +317,10 @@ def ssd_kernels(C, T, report, dev):
                 pos = torch.full((R,), n + 77, device=dev, dtype=torch.int32)
                 s = T(lambda: C.bias_decode(q, k, ring, pos, bias, dim=D, scale=0.09))
                 report(f"biased decode B{R} len{n} {H}q/{Hk}kv d{D} (keys only)", s, R * n * Hk * D * 2, 0)
+                if n == 1024:
+                    for sp in (1, 2, 4, 8):
+                        s = T(lambda: C.bias_decode(q, k, ring, pos, bias, dim=D, scale=0.09, splits=sp))
+                        report(f"   {sp} ranges", s, R * n * Hk * D * 2, 0)
                 kc, vc = ring.view(R, n, Hk, D), rnd(R, n, Hk, D)
                 ln = torch.full((R,), n, device=dev, dtype=torch.int32)
                 s = T(lambda: C.decode_attention(q.view(R, H, D), kc, vc, ln, scale=0.09))

@@ -282,7 +282,7 @@ struct SsmStepArgs {
   const float* dt_bias; const float* A_log; const float* D;
   void* ring; float* state;                        // [B, K, C] inputs by position % K; [B, H, N, P]
   const int* kv_len; const unsigned char* active;  // positions; null or 0 for rows that do not move
-  void* y; int B, H, P, N, G, K, C;
+  void* y; int B, H, P, N, G, K, C; int* status;
 };
 const char* ssm_step(const SsmStepArgs& a, cudaStream_t s);
 const char* gated_group_norm(int dtype, const void* y, long long ld_y, const void* z, long long ld_z, const float* w, void* out, long long rows,
@@ -311,7 +311,7 @@ struct BiasDecodeArgs {
 const char* bias_decode_any(const BiasDecodeArgs& a, cudaStream_t s);
 bool bias_decode_tc_supported(const BiasDecodeArgs& a);               // csrc/kernels/bias_decode_tc.cu
 int bias_decode_splits(const BiasDecodeArgs& a, int num_sms);
-const char* bias_decode_tc(const BiasDecodeArgs& a, int n_splits, cudaStream_t s);
+const char* bias_decode_tc(const BiasDecodeArgs& a, int n_splits, int* status, cudaStream_t s);
 
 // ---- flash attention (prefill / training) ----
 struct FlashArgs {

@@ -1406,6 +1406,7 @@ Tensor ssm_step(const Tensor& x, const Tensor& dtr, const Tensor& conv_w, const 
   a.ring = ring.data_ptr(); a.state = S.data_ptr<float>(); a.kv_len = kv_len.data_ptr<int>();
   Tensor y = out_empty({a.B, static_cast<int64_t>(a.H) * a.P}, x.options());
   a.y = y.data_ptr();
+  a.status = status_word();
   FERRL_CHECK(ferrl::ssm_step(a, stream()));
   return y;
 }
@@ -1475,7 +1476,7 @@ Tensor bias_decode(const Tensor& q, const Tensor& k, Tensor cache, const Tensor&
       ws = out_empty({static_cast<int64_t>(a.B) * heads * n * (dim + 2)}, q.options().dtype(at::kFloat));
       a.ws = ws.data_ptr<float>();
     }
-    FERRL_CHECK(ferrl::bias_decode_tc(a, n, stream()));
+    FERRL_CHECK(ferrl::bias_decode_tc(a, n, status_word(), stream()));
     return out;
   }
   FERRL_CHECK(ferrl::bias_decode_any(a, stream()));

@@ -21,6 +21,7 @@
 
 #include "../api.h"
 #include "../common.cuh"
+#include "../gemm/tc_common.cuh"
 #include "vec.cuh"
 
 namespace ferrl {
@@ -263,49 +264,65 @@ const char* launch_scan_n(const SsmScanArgs& a, cudaStream_t s) {
 }
 
 // ------------------------------------------------------------------------------------------------ one token
-// One CTA per (head, row).  Thread (rg, cg) walks rows rg, rg + RG, ... of S at columns cg * V .. cg * V + V - 1; kAhead
-// rows are requested before any is used.
-constexpr int kAhead = 8;
-template <typename T, int V>
-__global__ void __launch_bounds__(256) ssm_step_kernel(SsmStepArgs a) {
-  extern __shared__ __align__(16) float sm[];
-  pdl_trigger();
-  const int h = blockIdx.x, b = blockIdx.y;
-  const int rep = a.H / a.G, g = h / rep, inner = a.H * a.P;
-  float* sx = sm;                                   // [P rounded up to 4]
-  float* sB = sx + (a.P + 3) / 4 * 4;               // [N]
-  float* sC = sB + a.N;                             // [N]
-  float* part = sC + (2 * a.N + 3) / 4 * 4 - a.N;   // [RG][P]
+// One CTA per (head, row).  BULK: the head's matrix is fetched with one bulk copy while the convolution runs, updated in
+// shared memory and written back with another, so that several CTAs keep a streaming multiprocessor's memory requests in
+// flight without holding them in registers; otherwise it is updated in place in global memory.
+constexpr int kStepThreads = 128;
+struct StepSmem { int x, B, C, part, bar, bytes, RG; };      // offsets in floats behind the matrix, total bytes
+__host__ __device__ inline StepSmem step_smem(int P, int N, int V, bool bulk) {
+  StepSmem m;
+  m.RG = kStepThreads / (P / V) > 1 ? kStepThreads / (P / V) : 1;
+  m.x = bulk ? N * P : 0;
+  m.B = m.x + (P + 3) / 4 * 4;
+  m.C = m.B + N;
+  m.part = m.B + (2 * N + 3) / 4 * 4;
+  m.bar = m.part + (m.RG * P + 3) / 4 * 4;
+  m.bytes = m.bar * 4 + 16;
+  return m;
+}
+
+template <typename T, int V, bool BULK>
+__global__ void __launch_bounds__(kStepThreads) ssm_step_kernel(SsmStepArgs a) {
+  extern __shared__ __align__(128) float sm[];
   __shared__ float s_dt;
-  const int cgn = a.P / V, RG = max(1, 256 / cgn);
+  pdl_trigger();
+  const StepSmem lay = step_smem(a.P, a.N, V, BULK);
+  const int h = blockIdx.x, b = blockIdx.y;
+  const int rep = a.H / a.G, g = h / rep, inner = a.H * a.P, cgn = a.P / V;
+  float *sx = sm + lay.x, *sB = sm + lay.B, *sC = sm + lay.C, *part = sm + lay.part;
+  uint64_t* bar = reinterpret_cast<uint64_t*>(sm + lay.bar);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(bar + 1);
+  float* Sg = a.state + (static_cast<long long>(b) * a.H + h) * a.N * a.P;
   pdl_wait();
   T* y = static_cast<T*>(a.y) + static_cast<long long>(b) * inner + static_cast<long long>(h) * a.P;
   if (a.active && !a.active[b]) {                   // a retired row: nothing of its state moves
-    for (int i = threadIdx.x; i < a.P; i += 256) y[i] = from_f<T>(0.f);
+    for (int i = threadIdx.x; i < a.P; i += kStepThreads) y[i] = from_f<T>(0.f);
     return;
   }
-  // the first rows of the state are requested before the convolution needs its inputs
-  float* S = a.state + (static_cast<long long>(b) * a.H + h) * a.N * a.P;
-  const int rg0 = static_cast<int>(threadIdx.x) / cgn, c_0 = (static_cast<int>(threadIdx.x) - rg0 * cgn) * V;
-  Vec<V> v[kAhead];
-  if (static_cast<int>(threadIdx.x) < RG * cgn) {
-#pragma unroll
-    for (int k = 0; k < kAhead; ++k)
-      if (rg0 + k * RG < a.N) v[k] = ld<V>(S + static_cast<long long>(rg0 + k * RG) * a.P + c_0);
+  if constexpr (BULK) {
+    if (threadIdx.x == 0) {
+      tc::mbar_init(bar, 1);
+      *abort_flag = 0;
+      asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+      tc::mbar_expect_tx(bar, a.N * a.P * 4);
+      tc::bulk_load(sm, Sg, a.N * a.P * 4, bar);
+    }
   }
   const long long pos = a.kv_len[b];
   const int cur = static_cast<int>(pos % a.K);
   const T* xr = static_cast<const T*>(a.x) + b * a.ld_x;            // this token's [x | B | C] channels
   T* ring = static_cast<T*>(a.ring) + static_cast<long long>(b) * a.K * a.C;
   const int n_ch = a.P + 2 * a.N;
-  for (int i = threadIdx.x; i < n_ch; i += 256) {
+#pragma unroll 2
+  for (int i = threadIdx.x; i < n_ch; i += kStepThreads) {
     const int c = i < a.P ? h * a.P + i : (i < a.P + a.N ? inner + g * a.N + (i - a.P) : inner + a.G * a.N + g * a.N + (i - a.P - a.N));
     const T now = xr[c];
     float acc = a.conv_b ? a.conv_b[c] : 0.f;
+#pragma unroll 4
     for (int j = 1; j < a.K; ++j) {                 // token pos - j sits j slots behind the current one
-      if (j > pos) break;
       const int slot = cur - j < 0 ? cur - j + a.K : cur - j;
-      acc += a.conv_w[static_cast<long long>(c) * a.K + a.K - 1 - j] * to_f(ring[static_cast<long long>(slot) * a.C + c]);
+      const float past = j <= pos ? to_f(ring[static_cast<long long>(slot) * a.C + c]) : 0.f;
+      acc += a.conv_w[static_cast<long long>(c) * a.K + a.K - 1 - j] * past;
     }
     acc += a.conv_w[static_cast<long long>(c) * a.K + a.K - 1] * to_f(now);
     if (i < a.P || h == g * rep) ring[static_cast<long long>(cur) * a.C + c] = now;
@@ -317,52 +334,66 @@ __global__ void __launch_bounds__(256) ssm_step_kernel(SsmStepArgs a) {
   if (threadIdx.x == 0) s_dt = softplus_f(to_f(static_cast<const T*>(a.dt)[b * a.ld_dt + h]) + a.dt_bias[h]);
   __syncthreads();
   const float dt = s_dt, da = __expf(-__expf(a.A_log[h]) * dt);
-  for (int item = threadIdx.x; item < RG * cgn; item += 256) {
-    const int rg = item / cgn, c = (item - rg * cgn) * V;
-    Vec<V> acc, dx = ld<V>(sx + c);
+  bool ok = true;
+  if constexpr (BULK) ok = tc::mbar_wait(bar, 0, abort_flag, a.status, kStatusWaitTimeoutProducer);
+  float* S = BULK ? sm : Sg;
+  if (ok) {
+    for (int item = threadIdx.x; item < lay.RG * cgn; item += kStepThreads) {
+      const int rg = item / cgn, c = (item - rg * cgn) * V;
+      Vec<V> acc, dx = ld<V>(sx + c);
 #pragma unroll
-    for (int e = 0; e < V; ++e) { acc.v[e] = 0.f; dx.v[e] *= dt; }
-    for (int n0 = rg; n0 < a.N; n0 += RG * kAhead) {
-      if (n0 != rg || item != static_cast<int>(threadIdx.x)) {
+      for (int e = 0; e < V; ++e) { acc.v[e] = 0.f; dx.v[e] *= dt; }
+#pragma unroll 4
+      for (int n = rg; n < a.N; n += lay.RG) {
+        Vec<V> v = ld<V>(S + static_cast<long long>(n) * a.P + c);
+        const float bn = sB[n], cn = sC[n];
 #pragma unroll
-        for (int k = 0; k < kAhead; ++k)
-          if (n0 + k * RG < a.N) v[k] = ld<V>(S + static_cast<long long>(n0 + k * RG) * a.P + c);
-      }
-#pragma unroll
-      for (int k = 0; k < kAhead; ++k) {
-        const int n = n0 + k * RG;
-        if (n < a.N) {
-          const float bn = sB[n], cn = sC[n];
-#pragma unroll
-          for (int e = 0; e < V; ++e) {
-            v[k].v[e] = v[k].v[e] * da + bn * dx.v[e];
-            acc.v[e] += v[k].v[e] * cn;
-          }
-          st<V>(S + static_cast<long long>(n) * a.P + c, v[k]);
+        for (int e = 0; e < V; ++e) {
+          v.v[e] = v.v[e] * da + bn * dx.v[e];
+          acc.v[e] += v.v[e] * cn;
         }
+        st<V>(S + static_cast<long long>(n) * a.P + c, v);
       }
+      st<V>(part + rg * a.P + c, acc);
     }
-    st<V>(part + rg * a.P + c, acc);
+    if constexpr (BULK) tc::fence_async_smem();     // the bulk copy below reads what these threads wrote
   }
-  __syncthreads();
-  for (int i = threadIdx.x; i < a.P; i += 256) {
+  if (__syncthreads_or(!ok)) {
+    if constexpr (BULK) {
+      for (int i = 0; i < 64; ++i) __nanosleep(10000);   // let the copy in flight land before shared memory goes away
+    }
+    return;
+  }
+  if constexpr (BULK) {
+    if (threadIdx.x == 0) tc::bulk_store(Sg, sm, a.N * a.P * 4);
+  }
+  for (int i = threadIdx.x; i < a.P; i += kStepThreads) {
     float o = 0.f;
-    for (int r = 0; r < RG; ++r) o += part[r * a.P + i];
+    for (int r = 0; r < lay.RG; ++r) o += part[r * a.P + i];
     y[i] = from_f<T>(o + a.D[h] * sx[i]);
+  }
+  if constexpr (BULK) {
+    if (threadIdx.x == 0) tc::bulk_store_drain();
   }
 }
 
-template <typename T, int V>
+template <typename T, int V, bool BULK>
 const char* launch_step(const SsmStepArgs& a, cudaStream_t s) {
-  const int RG = std::max(1, 256 / (a.P / V));
-  const size_t smem = (static_cast<size_t>((a.P + 3) / 4 * 4) + (2 * a.N + 3) / 4 * 4 + static_cast<size_t>(RG) * a.P) * 4;
-  if (smem > 200 * 1024) return "ssm_step: head too large";
-  auto k = ssm_step_kernel<T, V>;
-  if (!FERRL_ONCE_PER_DEVICE(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) == cudaSuccess))
+  const int bytes = step_smem(a.P, a.N, V, BULK).bytes;
+  if (bytes > 226 * 1024) return "ssm_step: head too large";
+  auto k = ssm_step_kernel<T, V, BULK>;
+  if (!FERRL_ONCE_PER_DEVICE(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024) == cudaSuccess))
     return "ssm_step: cannot reserve shared memory";
-  launch_pdl(k, dim3(a.H, a.B), dim3(256), smem, s, a);
+  launch_pdl(k, dim3(a.H, a.B), dim3(kStepThreads), bytes, s, a);
   count_launch();
   return cudaGetLastError() == cudaSuccess ? nullptr : "ssm_step launch failed";
+}
+template <typename T>
+const char* launch_step_any(const SsmStepArgs& a, cudaStream_t s) {
+  if (a.P % 4 || (reinterpret_cast<uintptr_t>(a.state) & 15)) return launch_step<T, 1, false>(a, s);
+  // a bulk-staged matrix should leave room for a few CTAs on an SM
+  if (step_smem(a.P, a.N, 4, true).bytes <= 72 * 1024) return launch_step<T, 4, true>(a, s);
+  return launch_step<T, 4, false>(a, s);
 }
 
 // ------------------------------------------------------------------------------------------------ gated norm
@@ -442,9 +473,7 @@ const char* ssm_scan(const SsmScanArgs& a, cudaStream_t s) {
 
 const char* ssm_step(const SsmStepArgs& a, cudaStream_t s) {
   if (a.B == 0) return nullptr;
-  const bool vec = a.P % 4 == 0 && (reinterpret_cast<uintptr_t>(a.state) & 15) == 0;
-  if (a.dtype == kF32) return vec ? launch_step<float, 4>(a, s) : launch_step<float, 1>(a, s);
-  return vec ? launch_step<bf16, 4>(a, s) : launch_step<bf16, 1>(a, s);
+  return a.dtype == kF32 ? launch_step_any<float>(a, s) : launch_step_any<bf16>(a, s);
 }
 
 const char* gated_group_norm(int dtype, const void* y, long long ld_y, const void* z, long long ld_z, const float* w, void* out, long long rows,

@@ -56,7 +56,7 @@ ssm_scan_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constan
   uint8_t* sB = smem + kOffB;
   uint8_t* sX = smem + kOffX;
   uint8_t* sS = smem + kOffS;
-  float* s_vec = reinterpret_cast<float*>(smem + kOffVec);       // c_s - log2 dt_s
+  float* s_vec = reinterpret_cast<float*>(smem + kOffVec);       // log decay from s to the end of its 32 tokens + log2 dt_s
   float* s_sum = s_vec + kQ;                                     // log decay of each warp's tokens
   uint64_t* bars = reinterpret_cast<uint64_t*>(s_sum + 4);
   uint64_t *full = bars, *g_done = bars + 1, *s_done = bars + 2, *y_done = bars + 3, *u_done = bars + 4;
@@ -120,22 +120,27 @@ ssm_scan_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constan
     // ---- step sizes and log decays of the chunk
     const float z = raw + dtb;
     const float dt = raw == -INFINITY ? 0.f : (z > 20.f ? z : log1pf(__expf(z)));
-    float cum = A2 * dt;
+    // sums over this warp's 32 tokens: up to and with this one, and behind it; every exponent below is a sum of terms of
+    // one sign, so that a chunk's large total decay costs no accuracy between neighbours
+    float loc = A2 * dt, suf = __shfl_down_sync(0xffffffffu, loc, 1);
+    if (lane == 31) suf = 0.f;
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
-      const float v = __shfl_up_sync(0xffffffffu, cum, o);
-      if (lane >= o) cum += v;
+      const float u = __shfl_up_sync(0xffffffffu, loc, o), d = __shfl_down_sync(0xffffffffu, suf, o);
+      if (lane >= o) loc += u;
+      if (lane + o < 32) suf += d;
     }
-    if (lane == 31) s_sum[warp] = cum;
+    if (lane == 31) s_sum[warp] = loc;
     __syncthreads();
-    float last = 0.f;
+    float before = 0.f, after = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
       const float v = s_sum[w];
-      if (w < warp) cum += v;
-      last += v;
+      if (w < warp) before += v;
+      if (w > warp) after += v;
     }
-    s_vec[r] = cum - log2f(dt);                  // +inf where the token does not count
+    const float last = (s_sum[0] + s_sum[1]) + (s_sum[2] + s_sum[3]);
+    s_vec[r] = suf + log2f(dt);                  // -inf where the token does not count
     // ---- the state that enters: two bf16 terms for C S, and its decayed self as the accumulator of B^T X'
     if (c > 0) {
       const float dec = exp2f(last);
@@ -195,14 +200,25 @@ ssm_scan_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constan
         if (j <= warp) {
           tmem_ld32(tG + lane_sel + j * 32, v);
           tmem_ld_wait();
+          if (j < warp) {
+            float off = loc;                     // from the end of block j to this token
+            for (int w = j + 1; w < warp; ++w) off += s_sum[w];
+#pragma unroll
+            for (int e = 0; e < 16; ++e) {
+              const float2 bs = *reinterpret_cast<const float2*>(s_vec + j * 32 + 2 * e);
+              v[2 * e] = __float_as_uint(__uint_as_float(v[2 * e]) * exp2f(off + bs.x));
+              v[2 * e + 1] = __float_as_uint(__uint_as_float(v[2 * e + 1]) * exp2f(off + bs.y));
+            }
+          } else {                               // the diagonal block: the tokens are this warp's own
+#pragma unroll
+            for (int e = 0; e < 32; ++e) {
+              const float f = exp2f(loc - __shfl_sync(0xffffffffu, loc, e)) * __shfl_sync(0xffffffffu, dt, e);
+              v[e] = e > lane ? 0u : __float_as_uint(__uint_as_float(v[e]) * f);
+            }
+          }
 #pragma unroll
           for (int e = 0; e < 16; ++e) {
-            const float2 bs = *reinterpret_cast<const float2*>(s_vec + j * 32 + 2 * e);
-            float x = __uint_as_float(v[2 * e]) * exp2f(cum - bs.x), y = __uint_as_float(v[2 * e + 1]) * exp2f(cum - bs.y);
-            if (j == warp) {                     // the diagonal block
-              if (2 * e > lane) x = 0.f;
-              if (2 * e + 1 > lane) y = 0.f;
-            }
+            const float x = __uint_as_float(v[2 * e]), y = __uint_as_float(v[2 * e + 1]);
             m[e] = pair(x, y);
             const float2 f = unpair(m[e]);
             m[16 + e] = pair(x - f.x, y - f.y);
@@ -221,7 +237,7 @@ ssm_scan_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constan
       ok = __all_sync(0xffffffffu, ok);
       tc_fence_after();
       if (ok) {
-        const float f = exp2f(cum);
+        const float f = exp2f(before + loc);
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
           uint32_t v[32];
@@ -237,7 +253,7 @@ ssm_scan_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constan
     // G and C S have retired for every warp before C and S are overwritten
     if (__syncthreads_or(!ok)) { ok = false; break; }
     {
-      const float w = exp2f(last - cum) * dt;
+      const float w = exp2f(suf + after) * dt;
 #pragma unroll
       for (int k = 0; k < 8; ++k) {
         const int at = chunk_at(r, k);

@@ -230,15 +230,16 @@ bias_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     float* my_vec = s_vec + q * NH;
     float* my_cor = s_cor + q * NH;
     bool ok = true;
-    for (int i = 0; i < n_t; ++i) {
+    float bv[HP];                               // biases of this thread's slot, fetched a tile ahead
+    auto fetch = [&](int i) {
       const int slot = (t_lo + i) * kTok + r;
-      const bool live = slot < n;
-      float bv[HP];
-      {
-        const int d = live ? (cur >= slot ? cur - slot : cur - slot + a.slots) : 0;
+      const int d = slot < n ? (cur >= slot ? cur - slot : cur - slot + a.slots) : 0;
 #pragma unroll
-        for (int e = 0; e < HP; ++e) bv[e] = e < nh ? __ldg(bias + e * a.bias_ld + d) : 0.f;
-      }
+      for (int e = 0; e < HP; ++e) bv[e] = e < nh ? __ldg(bias + e * a.bias_ld + d) : 0.f;
+    };
+    if (n_t > 0) fetch(0);
+    for (int i = 0; i < n_t; ++i) {
+      const bool live = (t_lo + i) * kTok + r < n;
       if (!mbar_wait_warp(&s_full[i & 1], (i >> 1) & 1, abort_flag, geo.status, kStatusWaitTimeoutEpilogue)) { ok = false; break; }
       tc_fence_after();
       float sv[NH];
@@ -246,6 +247,7 @@ bias_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
       tmem_ld_wait();
 #pragma unroll
       for (int e = 0; e < HP; ++e) sv[e] = live ? sv[e] * c2 + bv[e] * kLog2e : -INFINITY;
+      if (i + 1 < n_t) fetch(i + 1);
       float* mx_buf = s_max + (i & 1) * 4 * HP;
       const float wm = lanes_reduce<HP, true>(sv, lane);
       if (lane < HP) mx_buf[q * HP + lane] = wm;

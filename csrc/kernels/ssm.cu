@@ -281,7 +281,8 @@ __host__ __device__ inline StepSmem step_smem(int P, int N, int V, bool bulk) {
   return m;
 }
 
-template <typename T, int V, bool BULK>
+// KT taps at compile time (the inputs of several channels are then requested together), or any number (KT = 0)
+template <typename T, int V, bool BULK, int KT>
 __global__ void __launch_bounds__(kStepThreads) ssm_step_kernel(SsmStepArgs a) {
   extern __shared__ __align__(128) float sm[];
   __shared__ float s_dt;
@@ -308,28 +309,54 @@ __global__ void __launch_bounds__(kStepThreads) ssm_step_kernel(SsmStepArgs a) {
       tc::bulk_load(sm, Sg, a.N * a.P * 4, bar);
     }
   }
-  const long long pos = a.kv_len[b];
-  const int cur = static_cast<int>(pos % a.K);
+  const int pos = a.kv_len[b];
+  const int cur = pos % a.K;
   const T* xr = static_cast<const T*>(a.x) + b * a.ld_x;            // this token's [x | B | C] channels
   T* ring = static_cast<T*>(a.ring) + static_cast<long long>(b) * a.K * a.C;
   const int n_ch = a.P + 2 * a.N;
-#pragma unroll 2
-  for (int i = threadIdx.x; i < n_ch; i += kStepThreads) {
-    const int c = i < a.P ? h * a.P + i : (i < a.P + a.N ? inner + g * a.N + (i - a.P) : inner + a.G * a.N + g * a.N + (i - a.P - a.N));
-    const T now = xr[c];
-    float acc = a.conv_b ? a.conv_b[c] : 0.f;
-#pragma unroll 4
-    for (int j = 1; j < a.K; ++j) {                 // token pos - j sits j slots behind the current one
-      const int slot = cur - j < 0 ? cur - j + a.K : cur - j;
-      const float past = j <= pos ? to_f(ring[static_cast<long long>(slot) * a.C + c]) : 0.f;
-      acc += a.conv_w[static_cast<long long>(c) * a.K + a.K - 1 - j] * past;
-    }
-    acc += a.conv_w[static_cast<long long>(c) * a.K + a.K - 1] * to_f(now);
+  auto channel = [&](int i) {
+    return i < a.P ? h * a.P + i : (i < a.P + a.N ? inner + g * a.N + (i - a.P) : inner + a.G * a.N + g * a.N + (i - a.P - a.N));
+  };
+  auto put = [&](int i, int c, T now, float acc) {
     if (i < a.P || h == g * rep) ring[static_cast<long long>(cur) * a.C + c] = now;
-    const float u = to_f(from_f<T>(silu_f(acc)));   // rounded as the convolution of whole sequences stores it
-    if (i < a.P) sx[i] = u;
-    else if (i < a.P + a.N) sB[i - a.P] = u;
-    else sC[i - a.P - a.N] = u;
+    sx[i < a.P ? i : i + lay.B - lay.x - a.P] = to_f(from_f<T>(silu_f(acc)));   // rounded as the convolution of whole sequences stores it
+  };
+  // token pos - j sits j slots behind the current one
+  auto slot = [&](int j) { return static_cast<long long>(cur - j < 0 ? cur - j + a.K : cur - j) * a.C; };
+  if constexpr (KT > 0) {
+    constexpr int CH = 3;
+    for (int i0 = threadIdx.x; i0 < n_ch; i0 += CH * kStepThreads) {
+      T now[CH], past[CH][KT - 1];
+      float w[CH][KT], acc[CH];
+#pragma unroll
+      for (int u = 0; u < CH; ++u) {
+        const int i = i0 + u * kStepThreads, c = channel(i < n_ch ? i : i0);
+        now[u] = xr[c];
+        acc[u] = a.conv_b ? a.conv_b[c] : 0.f;
+#pragma unroll
+        for (int j = 0; j < KT; ++j) w[u][j] = a.conv_w[static_cast<long long>(c) * KT + j];
+#pragma unroll
+        for (int j = 1; j < KT; ++j) past[u][j - 1] = ring[slot(j) + c];
+      }
+#pragma unroll
+      for (int u = 0; u < CH; ++u) {
+        const int i = i0 + u * kStepThreads;
+        if (i >= n_ch) break;
+#pragma unroll
+        for (int j = KT - 1; j >= 1; --j) acc[u] += w[u][KT - 1 - j] * (j <= pos ? to_f(past[u][j - 1]) : 0.f);
+        acc[u] += w[u][KT - 1] * to_f(now[u]);
+        put(i, channel(i), now[u], acc[u]);
+      }
+    }
+  } else {
+    for (int i = threadIdx.x; i < n_ch; i += kStepThreads) {
+      const int c = channel(i);
+      const T now = xr[c];
+      float acc = a.conv_b ? a.conv_b[c] : 0.f;
+      for (int j = 1; j < a.K; ++j) acc += a.conv_w[static_cast<long long>(c) * a.K + a.K - 1 - j] * (j <= pos ? to_f(ring[slot(j) + c]) : 0.f);
+      acc += a.conv_w[static_cast<long long>(c) * a.K + a.K - 1] * to_f(now);
+      put(i, c, now, acc);
+    }
   }
   if (threadIdx.x == 0) s_dt = softplus_f(to_f(static_cast<const T*>(a.dt)[b * a.ld_dt + h]) + a.dt_bias[h]);
   __syncthreads();
@@ -377,16 +404,20 @@ __global__ void __launch_bounds__(kStepThreads) ssm_step_kernel(SsmStepArgs a) {
   }
 }
 
-template <typename T, int V, bool BULK>
-const char* launch_step(const SsmStepArgs& a, cudaStream_t s) {
+template <typename T, int V, bool BULK, int KT>
+const char* launch_step_taps(const SsmStepArgs& a, cudaStream_t s) {
   const int bytes = step_smem(a.P, a.N, V, BULK).bytes;
   if (bytes > 226 * 1024) return "ssm_step: head too large";
-  auto k = ssm_step_kernel<T, V, BULK>;
+  auto k = ssm_step_kernel<T, V, BULK, KT>;
   if (!FERRL_ONCE_PER_DEVICE(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024) == cudaSuccess))
     return "ssm_step: cannot reserve shared memory";
   launch_pdl(k, dim3(a.H, a.B), dim3(kStepThreads), bytes, s, a);
   count_launch();
   return cudaGetLastError() == cudaSuccess ? nullptr : "ssm_step launch failed";
+}
+template <typename T, int V, bool BULK>
+const char* launch_step(const SsmStepArgs& a, cudaStream_t s) {
+  return a.K == 4 ? launch_step_taps<T, V, BULK, 4>(a, s) : launch_step_taps<T, V, BULK, 0>(a, s);
 }
 template <typename T>
 const char* launch_step_any(const SsmStepArgs& a, cudaStream_t s) {

@@ -48,6 +48,8 @@ def model_vocab_size(cfg: dict) -> int:
     """The model's vocabulary bound (nested ``text_config`` first): a positive integer, or the checkpoint is refused
     (crates/ferrl/src/hf.rs ``vocab_size_from_json``)."""
     raw = _preferred(cfg, "vocab_size")
+    if raw is None and cfg.get("model_type") is None and "architecture" in cfg:
+        raw = cfg.get("vocab")          # configurations dispatched on their architecture
     if isinstance(raw, bool) or not isinstance(raw, int) or raw <= 0:
         raise HfError(f"config vocab_size {raw!r} must be a positive integer")
     return raw

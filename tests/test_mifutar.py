@@ -615,8 +615,10 @@ def test_full_fine_tuning_reaches_every_tensor(tmp_path):
 # ------------------------------------------------------------------------------------------------ configuration, replay
 def test_configuration_is_read_and_checked(tmp_path):
     from ferrl_b200.models.loader import LoaderOpts, load_auto_policy
+    from ferrl_b200.hf import model_vocab_size
     from ferrl_b200.models.mifutar import mifutar_spec
     rows = {1: 8, 3: 8}
+    assert model_vocab_size(K.MIXED) == 89
     spec = mifutar_spec(K.MIXED, rows)
     assert [getattr(l.mixer, "window", None) for l in spec.layers] == [None, 7, None, 33] and spec.streams == 3 and spec.logit_scale == 0.5
     assert spec.layers[1].mlp is None and spec.layers[3].mlp.limit == 1.5 and spec.layers[3].mixer.scale == 0.5
